@@ -62,12 +62,15 @@ class PageMap:
 
     ``window`` (in positions) lets the map give back pages that no later query
     can reach; ``None`` keeps every page until the slot is released. ``keep_first``: the pages
-    that hold a sequence's first so many positions are never given back before that.
+    that hold a sequence's first so many positions are never given back before that. ``chunk``: no
+    later query reaches positions before the start of its own chunk of so many positions.
     """
 
-    def __init__(self, num_pages: int, window: Optional[int] = None, page_size: int = PAGE_SIZE, keep_first: int = 0):
+    def __init__(self, num_pages: int, window: Optional[int] = None, page_size: int = PAGE_SIZE, keep_first: int = 0,
+                 chunk: Optional[int] = None):
         self.page_size = page_size
         self.window = window
+        self.chunk = chunk
         self.keep_first = max(0, int(keep_first or 0))
         self.pool = FreeList(num_pages, "page")
         self._pages: Dict[int, List[int]] = {}     # slot -> page id per block of positions (-1: given back)
@@ -95,10 +98,12 @@ class PageMap:
 
     def trim(self, slot: int, length: int) -> None:
         """After a step that left ``slot`` at ``length``: give back the pages whose
-        positions all lie before the window of the next query (position ``length``)."""
-        if self.window is None:
+        positions all lie before the window (or the chunk) of the next query (position ``length``)."""
+        if self.window is None and self.chunk is None:
             return
-        first_needed = length - self.window + 1
+        first_needed = length - self.window + 1 if self.window is not None else 0
+        if self.chunk is not None:
+            first_needed = max(first_needed, length // self.chunk * self.chunk)
         pages = self._pages[slot]
         kept = -(-self.keep_first // self.page_size)          # blocks that hold the positions kept for good
         for block in range(kept, min(len(pages), max(0, first_needed) // self.page_size)):

@@ -29,11 +29,13 @@ from .pages import PAGE_SIZE, FreeList, PageMap
 @dataclass(frozen=True)
 class KVRequest:
     """Keys and values of every position (or of a window of positions) of a sequence. ``keep_first``: with a window,
-    the pages that hold a sequence's first so many positions are kept as well."""
+    the pages that hold a sequence's first so many positions are kept as well. ``chunk``: queries see keys of their own
+    chunk of so many positions only (counted from the sequence's start), so pages of finished chunks go back."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -49,6 +51,14 @@ class StateRequest:
     """A block of fixed shape per sequence, zero at the sequence's start."""
     shape: Tuple[int, ...]
     dtype: torch.dtype = torch.float32
+
+
+def keeps_state(request) -> bool:
+    """Whether a run with this request keeps a state that a step changes in place (running a step twice would change
+    it twice), by itself or as a member of a bundle."""
+    if isinstance(request, BundleRequest):
+        return any(keeps_state(m) for m in request.members)
+    return isinstance(request, StateRequest) or (isinstance(request, tuple) and bool(request))
 
 
 @dataclass(frozen=True)
@@ -76,7 +86,8 @@ class KVGroup:
     def __init__(self, request, runs: Sequence[int], num_pages: int, dtype: torch.dtype, device):
         self.request = request
         self.runs = list(runs)
-        self.pages = PageMap(num_pages, window=request.window, keep_first=getattr(request, "keep_first", 0))
+        self.pages = PageMap(num_pages, window=request.window, keep_first=getattr(request, "keep_first", 0),
+                             chunk=getattr(request, "chunk", None))
         if isinstance(request, RowsRequest):
             page_shape = (PAGE_SIZE, request.width)
         else:

@@ -8,8 +8,9 @@ from .ramupel import RamupelConfig
 from .botuvik import BotuvikConfig
 from .zasitar import ZasitarConfig
 from .dopuvik import DopuvikConfig
+from .vomotar import VomotarConfig
 
 __all__ = [
-    "ArchitectureConfig", "BotuvikConfig", "DopuvikConfig", "LlamaConfig", "RamupelConfig", "ZasitarConfig", "config_class_for", "config_from_dict",
+    "ArchitectureConfig", "BotuvikConfig", "DopuvikConfig", "LlamaConfig", "RamupelConfig", "VomotarConfig", "ZasitarConfig", "config_class_for", "config_from_dict",
     "known_architectures", "load_config", "register_architecture", "unregister_architecture",
 ]

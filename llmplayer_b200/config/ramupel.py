@@ -45,6 +45,10 @@ def _need(raw: dict, key: str, kind, where: str):
         if not isinstance(value, dict):
             raise ConfigError(f"{where}{key} must be an object, got {value!r}")
         return value
+    if kind is list:
+        if not isinstance(value, list):
+            raise ConfigError(f"{where}{key} must be a list, got {value!r}")
+        return value
     if kind is str:
         if not isinstance(value, str):
             raise ConfigError(f"{where}{key} must be a string, got {value!r}")

@@ -148,7 +148,22 @@ struct ScoreExtras {
     float scale_over_cap;
     const float* sinks;
     int keep;          // with a window: a sequence's first `keep` tokens stay visible to every later query (prompt kernels)
+    int chunk;         // > 0: a query at position p sees the keys of its own chunk of so many positions only (from p / chunk * chunk on)
+    // A distance bias per head (float32 [H] each, or both null): the score of the key n positions back loses
+    // dist_scale[h] * ln(1 + dist_rate[h] * n).
+    const float* dist_scale;
+    const float* dist_rate;
 };
+// the first position that a query at `pos` sees: by the window, by its chunk (the later of the two)
+__device__ __forceinline__ int first_seen(int pos, int window, const ScoreExtras& x) {
+    int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    if (x.chunk > 0) lo = max(lo, pos / x.chunk * x.chunk);
+    return lo;
+}
+// the distance bias in log2 units (scores are kept in log2 units: scale * ln(1 + r n) * log2(e) = scale * log2(1 + r n))
+__device__ __forceinline__ float distance_bias(float scale, float rate, int distance) {
+    return scale * __log2f(fmaf(rate, (float)max(distance, 0), 1.0f));
+}
 // tanh from the hardware's exp2 and a fast division: absolute error of about 1e-7
 __device__ __forceinline__ float lp_tanh_exp2(float x) {
     const float e = exp2f(x * 2.885390081777927f);
@@ -260,7 +275,7 @@ __device__ __forceinline__ void attention_decode_unit(
     const int kw = warp & 3, pg = warp >> 2;       // this warp's quarter of a page's keys, and its page of a group
     const int len = kv_len[b];
     const int pos = len - 1;                       // a length of zero or less is an empty sequence: no page is
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;      // read, nothing is stored, the output is zero
+    const int lo = first_seen(pos, window, fused.score);           // read, nothing is stored, the output is zero
     // Which pages this share takes. Fixed (min_share_pages == 0): share s takes pages s * pages_per_split ... of the
     // table. Fitted to the sequence (min_share_pages > 0): the pages that the sequence really has (within its
     // window) are cut into as many shares as leaves each at least min_share_pages, at most num_splits; the other
@@ -455,6 +470,13 @@ __device__ __forceinline__ void attention_decode_unit(
 #pragma unroll
     for (int i = 0; i < KSTEPS; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m0 = NEG_BIG, m1 = NEG_BIG, l0 = 0.f, l1 = 0.f;       // running maximum and sum of heads 2 t4 and 2 t4 + 1
+    const bool biased = SPLIT && fused.score.dist_scale != nullptr;
+    float ds0 = 0.f, ds1 = 0.f, dr0 = 0.f, dr1 = 0.f;            // the two heads' distance bias
+    if (biased) {
+        const int ha = head0 + min(2 * t4, nrows - 1), hb = head0 + min(2 * t4 + 1, nrows - 1);
+        ds0 = fused.score.dist_scale[ha]; dr0 = fused.score.dist_rate[ha];
+        ds1 = fused.score.dist_scale[hb]; dr1 = fused.score.dist_rate[hb];
+    }
 
     const int ngroups = (npages + PG - 1) / PG;
     const int new_at = new_page_at - page_lo;        // which of the share's pages holds the new token
@@ -508,6 +530,11 @@ __device__ __forceinline__ void attention_decode_unit(
                 s[1] = out_a ? NEG_BIG : shaped_score(s[1], scale_log2, fused.score);
                 s[2] = out_b ? NEG_BIG : shaped_score(s[2], scale_log2, fused.score);
                 s[3] = out_b ? NEG_BIG : shaped_score(s[3], scale_log2, fused.score);
+                if (biased) {
+                    const int na = pos - key_a, nb = pos - key_b;
+                    s[0] -= distance_bias(ds0, dr0, na); s[1] -= distance_bias(ds1, dr1, na);
+                    s[2] -= distance_bias(ds0, dr0, nb); s[3] -= distance_bias(ds1, dr1, nb);
+                }
                 float mx0 = fmaxf(s[0], s[2]), mx1 = fmaxf(s[1], s[3]);        // over the 16 keys: the lanes of equal t4
 #pragma unroll
                 for (int sh = 4; sh < 32; sh <<= 1) {

@@ -36,6 +36,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
                          float scale_log2, int window, ScoreExtras extras) {
     constexpr int KSTEPS = HD_MAX / 16;
     extern __shared__ __align__(128) uint8_t smem[];
+    __shared__ float bias_row[SPLIT ? 64 + PAGE : 1];      // the distance bias of a tile of rows and a page of keys, by row - key + 63
     lp_grid_release();
     lp_grid_wait();
     const int b = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
@@ -48,7 +49,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
     const int row0 = tile * 64;                         // first query row of this CTA among the new tokens
     const int rows = min(64, n_new - row0);
     const int first_pos = pos0 + row0, last_pos = pos0 + row0 + rows - 1;
-    const int lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+    const int lo = first_seen(first_pos, window, extras);
     const int page_lo = lo / PAGE, page_hi = last_pos / PAGE;
     // a window that keeps a sequence's first tokens visible: the pages that hold them (and lie before the window's
     // pages) are visited first; page number of the v-th visited page:
@@ -79,11 +80,17 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
     const int pos_lo = first_pos + min(r_lo, rows - 1), pos_hi = first_pos + min(r_hi, rows - 1);
     const int warp_last_pos = first_pos + min(warp * 16 + 15, rows - 1);
     const int warp_first_pos = first_pos + min(warp * 16, rows - 1);
+    // the first positions that the lane's two rows, and the warp's first and last row, see
+    const int low_lo = first_seen(pos_lo, window, extras), low_hi = first_seen(pos_hi, window, extras);
+    const int warp_first_low = first_seen(warp_first_pos, window, extras), warp_last_low = first_seen(warp_last_pos, window, extras);
 
     float o[KSTEPS * 2][4];
 #pragma unroll
     for (int i = 0; i < KSTEPS * 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_lo = NEG_BIG, m_hi = NEG_BIG, l_lo = 0.f, l_hi = 0.f;
+    const bool biased = SPLIT && extras.dist_scale != nullptr;
+    const float dist_scale = biased ? extras.dist_scale[h] : 0.f, dist_rate = biased ? extras.dist_rate[h] : 0.f;
+    const int row_lo = pos_lo - first_pos, row_hi = pos_hi - first_pos;
 
     load_page(smem, pages, table[page_of(0)], G, g, hd, tid, 128);
     cp_async_commit();
@@ -92,12 +99,13 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
         const int cur = vp & 1;
         if (vp + 1 < visited) load_page(smem + (cur ^ 1) * stage_bytes, pages, table[page_of(vp + 1)], G, g, hd, tid, 128);
         cp_async_commit();
+        const int key_base = p * PAGE;
+        if (SPLIT && biased) bias_row[tid] = distance_bias(dist_scale, dist_rate, first_pos - key_base + tid - (PAGE - 1));
         cp_async_wait<1>();
         __syncthreads();
-        const int key_base = p * PAGE;
         // pages wholly after this warp's rows, or wholly before their windows, contribute nothing
         const bool active = key_base <= warp_last_pos &&
-                            (window <= 0 || key_base + PAGE - 1 > warp_first_pos - window || key_base < keep);
+                            (key_base + PAGE - 1 >= warp_first_low || key_base < keep);
         if (active) {
             const uint32_t k_tile = smem_u32(smem + cur * stage_bytes);
             const uint32_t v_tile = k_tile + PAGE * hd * 2;
@@ -106,8 +114,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
             for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < 4; ++ks) scores_16keys<KSTEPS>(&s[ks * 2], qf, k_tile, ks * 16, hd, lane);
-            const bool edge = key_base + PAGE - 1 > warp_first_pos ||
-                              (window > 0 && key_base <= warp_last_pos - window);
+            const bool edge = key_base + PAGE - 1 > warp_first_pos || key_base < warp_last_low;
             float mx_lo = NEG_BIG, mx_hi = NEG_BIG;
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {
@@ -116,7 +123,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
                     const int key = key_base + nt * 8 + (lane & 3) * 2 + (e & 1);
                     const int pos = (e < 2) ? pos_lo : pos_hi;
                     float v = shaped_score(s[nt][e], scale_log2, extras);
-                    if (edge && (key > pos || (window > 0 && key <= pos - window && key >= keep))) v = NEG_BIG;
+                    if (SPLIT && biased) v -= bias_row[((e < 2) ? row_lo : row_hi) - (key - key_base) + PAGE - 1];
+                    if (edge && (key > pos || (key < ((e < 2) ? low_lo : low_hi) && key >= keep))) v = NEG_BIG;
                     s[nt][e] = v;
                     if (e < 2) mx_lo = fmaxf(mx_lo, v); else mx_hi = fmaxf(mx_hi, v);
                 }
@@ -179,7 +187,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
 // are computed once, the scale is folded into the exponent's FMA, exp2 is the hardware
 // approximation (relative error 2^-22, far below bfloat16's), and the tiles with the most keys
 // (the last ones of a prompt) are started first.
-template <int HD, int ROWS, bool SPLIT = false>
+// BIAS: scores lose a logarithm of the distance (ScoreExtras); the 127 values that a tile of rows and a page of keys can
+// need are formed once per page by the CTA's threads.
+template <int HD, int ROWS, bool SPLIT = false, bool BIAS = false>
 __global__ void __launch_bounds__(ROWS * 2, (SPLIT && HD <= 128) ? 3 : 1)
 attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out,
                                const __nv_bfloat16* __restrict__ pages, const int* __restrict__ page_table,
@@ -190,6 +200,7 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
     constexpr int TILE = PAGE * ROW;                  // bytes of a K (or V) tile
     constexpr int STAGE = 2 * TILE;
     extern __shared__ __align__(128) uint8_t smem[];
+    __shared__ float bias_row[BIAS ? ROWS + PAGE : 1];     // the distance bias of a tile of rows and a page of keys, by row - key + 63
     lp_grid_release();
     lp_grid_wait();
     const int b = blockIdx.z, h = blockIdx.y, tile = gridDim.x - 1 - blockIdx.x;
@@ -202,7 +213,7 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
     const int row0 = tile * ROWS;
     const int rows = min(ROWS, n_new - row0);
     const int first_pos = pos0 + row0, last_pos = pos0 + row0 + rows - 1;
-    const int lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+    const int lo = first_seen(first_pos, window, extras);
     const int page_lo = lo / PAGE, page_hi = last_pos / PAGE;
     // a window that keeps a sequence's first tokens visible: the pages that hold them (and lie before the window's
     // pages) are visited first; page number of the v-th visited page:
@@ -229,6 +240,9 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
     const int pos_lo = first_pos + min(r_lo, rows - 1), pos_hi = first_pos + min(r_hi, rows - 1);
     const int warp_last_pos = first_pos + min(warp * 16 + 15, rows - 1);
     const int warp_first_pos = first_pos + min(warp * 16, rows - 1);
+    // the first positions that the lane's two rows, and the warp's first and last row, see
+    const int low_lo = first_seen(pos_lo, window, extras), low_hi = first_seen(pos_hi, window, extras);
+    const int warp_first_low = first_seen(warp_first_pos, window, extras), warp_last_low = first_seen(warp_last_pos, window, extras);
 
     // byte offsets of this lane's ldmatrix rows inside a slice of 16 keys
     uint32_t k_off[KSTEPS], v_off[KSTEPS];
@@ -247,7 +261,10 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
     for (int i = 0; i < KSTEPS * 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_lo = NEG_BIG, m_hi = NEG_BIG, l_lo = 0.f, l_hi = 0.f;      // maxima in scaled log2 units
     const bool capped = extras.cap_log2 > 0.f;
-    const float scale_log2 = capped ? 1.0f : scale_log2_arg;
+    const float scale_log2 = (capped || BIAS) ? 1.0f : scale_log2_arg;
+    float dist_scale = 0.f, dist_rate = 0.f;
+    if constexpr (BIAS) { dist_scale = extras.dist_scale[h]; dist_rate = extras.dist_rate[h]; }
+    const int row_lo = pos_lo - first_pos, row_hi = pos_hi - first_pos;
 
     load_page(smem, pages, table[page_of(0)], G, g, HD, tid, ROWS * 2);
     cp_async_commit();
@@ -256,11 +273,14 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
         const int cur = vp & 1;
         if (vp + 1 < visited) load_page(smem + (cur ^ 1) * STAGE, pages, table[page_of(vp + 1)], G, g, HD, tid, ROWS * 2);
         cp_async_commit();
+        const int key_base = p * PAGE;
+        if constexpr (BIAS) {
+            if (tid < ROWS + PAGE) bias_row[tid] = distance_bias(dist_scale, dist_rate, first_pos - key_base + tid - (PAGE - 1));
+        }
         cp_async_wait<1>();
         __syncthreads();
-        const int key_base = p * PAGE;
         const bool active = key_base <= warp_last_pos &&
-                            (window <= 0 || key_base + PAGE - 1 > warp_first_pos - window || key_base < keep);
+                            (key_base + PAGE - 1 >= warp_first_low || key_base < keep);
         if (active) {
             const uint32_t k_tile = smem_u32(smem + cur * STAGE);
             const uint32_t v_tile = k_tile + TILE;
@@ -283,8 +303,17 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
 #pragma unroll
                     for (int e = 0; e < 4; ++e) s[nt][e] = shaped_score(s[nt][e], scale_log2_arg, extras);
             }
-            const bool edge = key_base + PAGE - 1 > warp_first_pos ||
-                              (window > 0 && key_base <= warp_last_pos - window);
+            if constexpr (BIAS) {         // the same with the distance bias taken off
+#pragma unroll
+                for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int key = nt * 8 + (lane & 3) * 2 + (e & 1);
+                        const float bias = bias_row[((e < 2) ? row_lo : row_hi) - key + PAGE - 1];
+                        s[nt][e] = capped ? s[nt][e] - bias : fmaf(s[nt][e], scale_log2_arg, -bias);
+                    }
+            }
+            const bool edge = key_base + PAGE - 1 > warp_first_pos || key_base < warp_last_low;
             if (edge) {
 #pragma unroll
                 for (int nt = 0; nt < 8; ++nt)
@@ -292,7 +321,7 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
                     for (int e = 0; e < 4; ++e) {
                         const int key = key_base + nt * 8 + (lane & 3) * 2 + (e & 1);
                         const int pos = (e < 2) ? pos_lo : pos_hi;
-                        if (key > pos || (window > 0 && key <= pos - window && key >= keep)) s[nt][e] = -INFINITY;
+                        if (key > pos || (key < ((e < 2) ? low_lo : low_hi) && key >= keep)) s[nt][e] = -INFINITY;
                     }
             }
             float mx_lo = -INFINITY, mx_hi = -INFINITY;
@@ -450,6 +479,13 @@ template <typename K> int set_smem(K kernel, int bytes, const char* what) {
     return 0;
 }
 
+int check_shaping(const char* what, int keep, int chunk, const float* dist_scale, const float* dist_rate, int split_weights) {
+    if ((dist_scale == nullptr) != (dist_rate == nullptr)) LP_REFUSE("%s: a distance bias has a scale and a rate per head", what);
+    if (dist_scale && !split_weights) LP_REFUSE("%s: a distance bias comes with weights at float32 precision", what);
+    if (keep > 0 && chunk > 0) LP_REFUSE("%s: kept first tokens (%d) and chunks (%d) exclude each other", what, keep, chunk);
+    return 0;
+}
+
 int check_geometry(const char* what, int H, int G, int hd) {
     if (H <= 0 || G <= 0 || H % G) LP_REFUSE("%s: %d query heads over %d key heads", what, H, G);
     if (hd < 16 || hd > 256 || hd % 16) LP_REFUSE("%s: head size %d (supported: multiples of 16 up to 256)", what, hd);
@@ -457,8 +493,13 @@ int check_geometry(const char* what, int H, int G, int hd) {
 }
 
 // softcap > 0: scores are capped at it; sinks: float32 [H] or null (see ScoreExtras)
-static ScoreExtras make_extras(float scale, float softcap, const float* sinks, int keep = 0) {
+// chunk > 0: keys of the query's own chunk only; dist_scale, dist_rate: float32 [H] each, or both null
+static ScoreExtras make_extras(float scale, float softcap, const float* sinks, int keep = 0, int chunk = 0,
+                               const float* dist_scale = nullptr, const float* dist_rate = nullptr) {
     ScoreExtras x{};
+    x.chunk = chunk > 0 ? chunk : 0;
+    x.dist_scale = dist_scale;
+    x.dist_rate = dist_rate;
     x.keep = keep > 0 ? keep : 0;
     if (softcap > 0.f) {
         x.cap_log2 = softcap * 1.4426950408889634f;
@@ -475,10 +516,13 @@ static ScoreExtras make_extras(float scale, float softcap, const float* sinks, i
 extern "C" int lp_attention_prefill(const void* q, void* out, const void* pages, const int* page_table, int pt_stride,
                                     const int* q_start, const int* kv_len, int B, int max_new, int H, int G, int hd,
                                     int page_size, float scale, int window, float softcap, const float* sinks,
-                                    int split_weights, int keep, cudaStream_t stream) {
+                                    int split_weights, int keep, int chunk, const float* dist_scale,
+                                    const float* dist_rate, cudaStream_t stream) {
     if (B <= 0 || max_new <= 0) return 0;
-    const ScoreExtras extras = make_extras(scale, softcap, sinks, keep);
+    const ScoreExtras extras = make_extras(scale, softcap, sinks, keep, chunk, dist_scale, dist_rate);
     int rc = check_geometry("attention_prefill", H, G, hd);
+    if (rc) return rc;
+    rc = check_shaping("attention_prefill", window > 0 ? keep : 0, chunk, dist_scale, dist_rate, split_weights);
     if (rc) return rc;
     if (page_size != PAGE) LP_REFUSE("attention_prefill: pages of %d positions (built for %d)", page_size, PAGE);
     if (H > 65535 || B > 65535) LP_REFUSE("attention_prefill: %d heads x %d sequences exceed the grid", H, B);
@@ -516,10 +560,15 @@ extern "C" int lp_attention_prefill(const void* q, void* out, const void* pages,
     } while (0)
 #define LP_PREFILL_EXACT_SPLIT(HD, ROWS)                                                                         \
     do {                                                                                                         \
-        rc = set_smem(attention_prefill_exact_kernel<HD, ROWS, true>, smem, "attention_prefill");                \
+        if (dist_scale) LP_PREFILL_EXACT_SHAPED(HD, ROWS, true);                                                 \
+        else LP_PREFILL_EXACT_SHAPED(HD, ROWS, false);                                                           \
+    } while (0)
+#define LP_PREFILL_EXACT_SHAPED(HD, ROWS, BIASED)                                                                \
+    do {                                                                                                         \
+        rc = set_smem(attention_prefill_exact_kernel<HD, ROWS, true, BIASED>, smem, "attention_prefill");        \
         if (rc) return rc;                                                                                       \
         dim3 grid_exact((max_new + ROWS - 1) / ROWS, H, B);                                                      \
-        lp_launch(attention_prefill_exact_kernel<HD, ROWS, true>, grid_exact, ROWS * 2, smem, stream,            \
+        lp_launch(attention_prefill_exact_kernel<HD, ROWS, true, BIASED>, grid_exact, ROWS * 2, smem, stream,    \
                   (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)pages, page_table,         \
                   pt_stride, q_start, kv_len, H, G, scale_log2, window, extras);                                 \
     } while (0)
@@ -529,6 +578,7 @@ extern "C" int lp_attention_prefill(const void* q, void* out, const void* pages,
         else if (hd <= 64) LP_PREFILL_SPLIT(64); else if (hd <= 96) LP_PREFILL_SPLIT(96); else if (hd <= 128) LP_PREFILL_SPLIT(128);
         else if (hd <= 192) LP_PREFILL_SPLIT(192); else LP_PREFILL_SPLIT(256);
 #undef LP_PREFILL_EXACT_SPLIT
+#undef LP_PREFILL_EXACT_SHAPED
 #undef LP_PREFILL_SPLIT
     }
     else if (hd == 64 && tall) LP_PREFILL_EXACT(64, 128);
@@ -555,12 +605,15 @@ extern "C" long long lp_attention_decode_scratch(int B, int H, int hd, int num_s
 static int attention_decode_launch(const void* q, void* out, const void* pages, const int* page_table, int pt_stride,
                                    const int* kv_len, float* scratch, int B, int H, int G, int hd, int page_size,
                                    float scale, int window, int pages_per_split, int num_splits, int min_share_pages,
-                                   float softcap, const float* sinks, int split_weights, cudaStream_t stream, int keep = 0) {
+                                   float softcap, const float* sinks, int split_weights, cudaStream_t stream, int keep = 0,
+                                   int chunk = 0, const float* dist_scale = nullptr, const float* dist_rate = nullptr) {
     if (B <= 0) return 0;
     if (keep > 0 && min_share_pages <= 0) LP_REFUSE("attention_decode: kept first tokens need shares fitted to the sequence (%d)", keep);
     FusedDecodeArgs plain_args{};
-    plain_args.score = make_extras(scale, softcap, sinks, window > 0 ? keep : 0);
+    plain_args.score = make_extras(scale, softcap, sinks, window > 0 ? keep : 0, chunk, dist_scale, dist_rate);
     int rc = check_geometry("attention_decode", H, G, hd);
+    if (rc) return rc;
+    rc = check_shaping("attention_decode", window > 0 ? keep : 0, chunk, dist_scale, dist_rate, split_weights);
     if (rc) return rc;
     if (page_size != PAGE) LP_REFUSE("attention_decode: pages of %d positions (built for %d)", page_size, PAGE);
     if (pages_per_split <= 0 || num_splits <= 0) LP_REFUSE("attention_decode: %d shares of %d pages", num_splits, pages_per_split);
@@ -617,12 +670,12 @@ extern "C" int lp_attention_decode(const void* q, void* out, const void* pages, 
 extern "C" int lp_attention_decode_fitted(const void* q, void* out, const void* pages, const int* page_table,
                                           int pt_stride, const int* kv_len, float* scratch, int B, int H, int G, int hd,
                                           int page_size, float scale, int window, int num_splits, int min_share_pages,
-                                          float softcap, const float* sinks, int split_weights, int keep,
-                                          cudaStream_t stream) {
+                                          float softcap, const float* sinks, int split_weights, int keep, int chunk,
+                                          const float* dist_scale, const float* dist_rate, cudaStream_t stream) {
     if (min_share_pages <= 0) LP_REFUSE("attention_decode_fitted: shares of at least %d pages", min_share_pages);
     return attention_decode_launch(q, out, pages, page_table, pt_stride, kv_len, scratch, B, H, G, hd, page_size, scale,
                                    window, pt_stride > 0 ? pt_stride : 1, num_splits, min_share_pages, softcap, sinks,
-                                   split_weights, stream, keep);
+                                   split_weights, stream, keep, chunk, dist_scale, dist_rate);
 }
 
 // Decode attention that starts from the fused projection output: rotation of queries and of the new key,

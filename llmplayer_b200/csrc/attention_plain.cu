@@ -22,7 +22,8 @@ __global__ void __launch_bounds__(KB)
 attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV* __restrict__ pages,
                        const int* __restrict__ page_table, int pt_stride, const int* __restrict__ seq_ids,
                        const int* __restrict__ positions, int H, int G, int hd, int page_size, float scale,
-                       int window, float softcap, const float* __restrict__ sinks, int keep) {
+                       int window, float softcap, const float* __restrict__ sinks, int keep, int chunk,
+                       const float* __restrict__ dist_scale, const float* __restrict__ dist_rate) {
     __shared__ float qs[MAX_HD];
     __shared__ float prob[KB];
     __shared__ long long row_off[KB];
@@ -32,7 +33,9 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
     const int g = h / (H / G);
     const int seq = seq_ids[t];
     const int pos = positions[t];
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);         // keys of the query's own chunk of positions only
+    const float ds = dist_scale ? dist_scale[h] : 0.f, dr = dist_scale ? dist_rate[h] : 0.f;
     // a window may keep a sequence's first `keep` tokens visible as well: keys [0, keep_end) besides [lo, pos]
     const int keep_end = keep < lo ? (keep > 0 ? keep : 0) : lo;
     const int c_lo = (lo / KB) * KB;
@@ -60,6 +63,7 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
             for (int i = 0; i < hd; ++i) dot = fmaf(qs[i], lp_to_float(kr[i]), dot);
             sc = dot * scale;
             if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+            if (dist_scale) sc -= ds * log1pf(dr * (float)(pos - key));
         }
         const float cmax = lp_block_max(sc, scratch);
         const float m_new = fmaxf(m, cmax);
@@ -104,12 +108,17 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
 // q, out: [T, H, hd]; pages: [num_pages, 2, G, page_size, hd]; page_table: [B, pt_stride];
 // seq_ids, positions: [T]. window <= 0: all keys up to the query's position. softcap > 0: a score s becomes
 // softcap * tanh(s / softcap) after the scale. sinks (optional): float32 [H], see the kernel. keep > 0 (with a window):
-// the sequence's first `keep` tokens stay visible to every later query, at their true positions.
+// the sequence's first `keep` tokens stay visible to every later query, at their true positions. chunk > 0: a query at p
+// sees keys from p / chunk * chunk on only. dist_scale, dist_rate (optional, float32 [H] each): a key n positions back
+// loses dist_scale[h] * ln(1 + dist_rate[h] * n) of its score.
 extern "C" int lp_attention_plain(const void* q, void* out, int q_dtype, const void* pages, int kv_dtype,
                                   const int* page_table, int pt_stride, const int* seq_ids, const int* positions,
                                   int T, int H, int G, int hd, int page_size, float scale, int window,
-                                  float softcap, const float* sinks, int keep, cudaStream_t stream) {
+                                  float softcap, const float* sinks, int keep, int chunk, const float* dist_scale,
+                                  const float* dist_rate, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if ((dist_scale == nullptr) != (dist_rate == nullptr)) LP_REFUSE("attention_plain: a distance bias has a scale and a rate per head");
+    if (keep > 0 && window > 0 && chunk > 0) LP_REFUSE("attention_plain: kept first tokens (%d) and chunks (%d) exclude each other", keep, chunk);
     if (H <= 0 || G <= 0 || H % G) LP_REFUSE("attention_plain: %d query heads over %d key heads", H, G);
     if (hd <= 0 || hd > MAX_HD) LP_REFUSE("attention_plain: head size %d (supported: 1..%d)", hd, MAX_HD);
     if (page_size <= 0) LP_REFUSE("attention_plain: page size %d", page_size);
@@ -118,7 +127,8 @@ extern "C" int lp_attention_plain(const void* q, void* out, int q_dtype, const v
 #define LP_LAUNCH_ATT(TQ, TKV)                                                                                 \
     attention_plain_kernel<TQ, TKV><<<grid, KB, 0, stream>>>((const TQ*)q, (TQ*)out, (const TKV*)pages,          \
                                                              page_table, pt_stride, seq_ids, positions, H, G,  \
-                                                             hd, page_size, scale, window, softcap, sinks, keep)
+                                                             hd, page_size, scale, window, softcap, sinks, keep, \
+                                                             chunk, dist_scale, dist_rate)
     if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_LAUNCH_ATT(float, float);
     else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_LAUNCH_ATT(__nv_bfloat16, __nv_bfloat16);
     else if (q_dtype == LP_F32 && kv_dtype == LP_BF16) LP_LAUNCH_ATT(float, __nv_bfloat16);

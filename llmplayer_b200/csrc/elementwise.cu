@@ -47,6 +47,13 @@ extern "C" int lp_embed(const void* table, int table_dtype, const int* tokens, f
 // in registers (up to PER * 256 values; wider rows take the two-pass kernel below).
 // `zero` (optional): a float32 buffer that the blocks clear on the side, for the product that
 // follows the norm and sums its partial results with atomics.
+// `parts` > 1: a row is cut into that many equal parts that are each divided by their own root mean square; a block then
+// handles one part (block r: part r % parts of row r / parts) and `d` is the width of a part.
+__device__ __forceinline__ long long norm_part(const int* rows, int parts, int& part) {
+    const int row = parts == 1 ? blockIdx.x : blockIdx.x / parts;
+    part = parts == 1 ? 0 : blockIdx.x - row * parts;
+    return (long long)(rows ? rows[row] : row) * parts + part;
+}
 constexpr int NORM_THREADS = 256;
 constexpr int NORM_PER = 16;
 
@@ -55,12 +62,14 @@ template <typename TOut, typename TAdd>
 __global__ void __launch_bounds__(NORM_THREADS)
 rmsnorm_kernel(float* __restrict__ x, const TAdd* __restrict__ add, const int* __restrict__ rows,
                const float* __restrict__ w, TOut* __restrict__ out, int d, float eps, float* __restrict__ zero,
-               long long zero_count) {
+               long long zero_count, int parts) {
     __shared__ float scratch[32];
     lp_grid_release();
     lp_grid_wait();
     const int r = blockIdx.x;
-    const long long src = rows ? rows[r] : r;
+    int part;
+    const long long src = norm_part(rows, parts, part);
+    w += (long long)part * d;
     float* xr = x + src * d;
     float v[NORM_PER];
     float ss = 0.f;
@@ -91,12 +100,15 @@ constexpr int NORM_VEC_PER = 4;          // float4 per thread: rows up to 256 * 
 template <typename TOut>
 __global__ void __launch_bounds__(NORM_THREADS)
 rmsnorm_vec4_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w,
-                    TOut* __restrict__ out, int d, float eps, float* __restrict__ zero, long long zero_count) {
+                    TOut* __restrict__ out, int d, float eps, float* __restrict__ zero, long long zero_count,
+                    int parts) {
     __shared__ float scratch[32];
     lp_grid_release();
     lp_grid_wait();
     const int r = blockIdx.x;
-    const long long src = rows ? rows[r] : r;
+    int part;
+    const long long src = norm_part(rows, parts, part);
+    w += (long long)part * d;
     const float4* xr = reinterpret_cast<const float4*>(x + src * d);
     const int quads = d >> 2;
     float4 v[NORM_VEC_PER];
@@ -136,12 +148,14 @@ template <typename TOut, typename TAdd>
 __global__ void rmsnorm_wide_kernel(float* __restrict__ x, const TAdd* __restrict__ add,
                                     const int* __restrict__ rows, const float* __restrict__ w,
                                     TOut* __restrict__ out, int d, float eps, float* __restrict__ zero,
-                                    long long zero_count) {
+                                    long long zero_count, int parts) {
     __shared__ float scratch[32];
     lp_grid_release();
     lp_grid_wait();
     const int r = blockIdx.x;
-    const long long src = rows ? rows[r] : r;
+    int part;
+    const long long src = norm_part(rows, parts, part);
+    w += (long long)part * d;
     float* xr = x + src * d;
     float ss = 0.f;
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
@@ -158,19 +172,23 @@ __global__ void rmsnorm_wide_kernel(float* __restrict__ x, const TAdd* __restric
 
 extern "C" int lp_rmsnorm(float* x, const void* add, int add_dtype, const int* rows, const float* w, void* out,
                           int out_dtype, int R, int d, float eps, float* zero, long long zero_count,
-                          cudaStream_t stream) {
+                          int parts, cudaStream_t stream) {
     if (R <= 0) return 0;
     if (d <= 0) LP_REFUSE("rmsnorm: width %d", d);
+    if (parts <= 0 || d % parts) LP_REFUSE("rmsnorm: rows of %d values in %d equal parts", d, parts);
+    if ((long long)R * parts > 2147483647LL) LP_REFUSE("rmsnorm: %d rows in %d parts exceed the grid", R, parts);
+    R *= parts;
+    d /= parts;
     if (add && rows) LP_REFUSE("rmsnorm: a fused residual add cannot be combined with a row selection");
     const bool wide = d > NORM_THREADS * NORM_PER;
     if (!add && d % 4 == 0 && d <= NORM_THREADS * 4 * NORM_VEC_PER &&
         ((((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0)) {
         if (out_dtype == LP_BF16)
             lp_launch(rmsnorm_vec4_kernel<__nv_bfloat16>, R, NORM_THREADS, 0, stream, (const float*)x, rows, w,
-                      (__nv_bfloat16*)out, d, eps, zero, zero_count);
+                      (__nv_bfloat16*)out, d, eps, zero, zero_count, parts);
         else if (out_dtype == LP_F32)
             lp_launch(rmsnorm_vec4_kernel<float>, R, NORM_THREADS, 0, stream, (const float*)x, rows, w, (float*)out, d,
-                      eps, zero, zero_count);
+                      eps, zero, zero_count, parts);
         else LP_REFUSE("rmsnorm: dtype code out=%d", out_dtype);
         return lp_check_launch("rmsnorm");
     }
@@ -178,10 +196,10 @@ extern "C" int lp_rmsnorm(float* x, const void* add, int add_dtype, const int* r
     do {                                                                                                        \
         if (wide)                                                                                               \
             lp_launch(rmsnorm_wide_kernel<TOUT, TADD>, R, 512, 0, stream, x, (const TADD*)add, rows, w,          \
-                      (TOUT*)out, d, eps, zero, zero_count);                                                    \
+                      (TOUT*)out, d, eps, zero, zero_count, parts);                                                    \
         else                                                                                                    \
             lp_launch(rmsnorm_kernel<TOUT, TADD>, R, NORM_THREADS, 0, stream, x, (const TADD*)add, rows, w,      \
-                      (TOUT*)out, d, eps, zero, zero_count);                                                    \
+                      (TOUT*)out, d, eps, zero, zero_count, parts);                                                    \
     } while (0)
     if (out_dtype == LP_F32 && add_dtype == LP_F32) LP_LAUNCH_NORM(float, float);
     else if (out_dtype == LP_F32 && add_dtype == LP_BF16) LP_LAUNCH_NORM(float, __nv_bfloat16);
@@ -625,7 +643,8 @@ extern "C" int lp_advance(int* tokens, int* positions, int* kv_len, const int* s
 // attention kernels see one head size; queries go to q_out[t, h, :hdp], keys and values to the page of the token's
 // sequence that holds its position, pages[page][0|1][g][position % page_size][:hdp]. A warp per head; all float32.
 // `qgain` / `kgain` (optional, [dk], shared by the heads): BEFORE the rotation every query / key head is RMS-normed
-// over dk with that gain and `gain_eps` inside the root. G = 0 with `pages` null: a layer that has queries only.
+// over dk with that gain and `gain_eps` inside the root. `vnorm`: every value head is divided by its root mean square over
+// dv (`vnorm_eps` inside the root). G = 0 with `pages` null: a layer that has queries only.
 constexpr int PREP_MAX = 256;
 template <typename TQ, typename TKV>
 __global__ void __launch_bounds__(256)
@@ -633,7 +652,8 @@ qkv_prepare_kernel(const float* __restrict__ qkv, int ld, const float* __restric
                    const int* __restrict__ positions, const int* __restrict__ seq_ids, const int* __restrict__ page_table,
                    int pt_stride, TQ* __restrict__ q_out, TKV* __restrict__ pages, int H, int G, int dk, int dv, int hdp,
                    int rd, int interleaved, int unit, float unit_eps, int page_size, float* __restrict__ zero,
-                   long long zero_count, const float* __restrict__ qgain, const float* __restrict__ kgain, float gain_eps) {
+                   long long zero_count, const float* __restrict__ qgain, const float* __restrict__ kgain, float gain_eps,
+                   int vnorm, float vnorm_eps) {
     __shared__ float cs[PREP_MAX];
     __shared__ float buf[8][PREP_MAX];
     lp_grid_release();
@@ -697,8 +717,17 @@ qkv_prepare_kernel(const float* __restrict__ qkv, int ld, const float* __restric
             const int g = item - H - G;
             const int src = (H + G) * dk + g * dv;
             TKV* dst = pages + (((page * 2 + 1) * G + g) * page_size + r) * hdp;
+            float factor = 1.0f;
+            if (vnorm) {
+                float ss = 0.f;
+                for (int e = lane; e < dv; e += 32) {
+                    const float val = row[src + e] + (bias ? bias[src + e] : 0.f);
+                    ss += val * val;
+                }
+                factor = 1.0f / sqrtf(lp_warp_sum(ss) / (float)dv + vnorm_eps);
+            }
             for (int e = lane; e < hdp; e += 32)
-                dst[e] = lp_from_float<TKV>(e < dv ? row[src + e] + (bias ? bias[src + e] : 0.f) : 0.f);
+                dst[e] = lp_from_float<TKV>(e < dv ? (row[src + e] + (bias ? bias[src + e] : 0.f)) * factor : 0.f);
         }
     }
 }
@@ -707,7 +736,8 @@ extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const
                               const int* seq_ids, const int* page_table, int pt_stride, void* q_out, int q_dtype,
                               void* pages, int kv_dtype, int T, int H, int G, int dk, int dv, int hdp, int rd,
                               int interleaved, int unit, float unit_eps, int page_size, float* zero, long long zero_count,
-                              const float* qgain, const float* kgain, float gain_eps, cudaStream_t stream) {
+                              const float* qgain, const float* kgain, float gain_eps, int vnorm, float vnorm_eps,
+                              cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || G < 0 || dk <= 0 || dv <= 0) LP_REFUSE("qkv_prepare: %d / %d heads of %d and %d", H, G, dk, dv);
     if (hdp < dk || hdp < dv || dk > PREP_MAX) LP_REFUSE("qkv_prepare: heads of %d and %d stored in %d (at most %d)", dk, dv, hdp, PREP_MAX);
@@ -719,7 +749,7 @@ extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const
 #define LP_LAUNCH_PREP(TQ, TKV)                                                                                       \
     lp_launch(qkv_prepare_kernel<TQ, TKV>, T, 256, 0, stream, qkv, ld, bias, inv_freq, positions, seq_ids, page_table, \
               pt_stride, (TQ*)q_out, (TKV*)pages, H, G, dk, dv, hdp, rd, interleaved, unit, unit_eps, page_size, zero,  \
-              zero_count, qgain, kgain, gain_eps)
+              zero_count, qgain, kgain, gain_eps, vnorm, vnorm_eps)
     if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_LAUNCH_PREP(float, float);
     else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_LAUNCH_PREP(__nv_bfloat16, __nv_bfloat16);
     else LP_REFUSE("qkv_prepare: dtype codes q=%d kv=%d", q_dtype, kv_dtype);
@@ -1040,4 +1070,96 @@ extern "C" int lp_scaled_sum(float* x, const float* a, const float* va, float sa
     if (blocks > 148 * 16) blocks = 148 * 16;
     lp_launch(scaled_sum_kernel, (unsigned)blocks, 256, 0, stream, x, a, va, sa, b, vb, sb, T, d);
     return lp_check_launch("scaled_sum");
+}
+
+// ---------------------------------------------------------------- two sublayers' results, each normed, then summed
+// x[t] += sa * a[t] / rms(a[t]) * wa + sb * b[t] / rms(b[t]) * wb with rms(v) = sqrt(mean(v^2) + eps) over the row, and,
+// when `w2` is given, out2[t] = the RMS norm of the new x[t] in `parts` equal parts (each divided by its own root mean
+// square, `eps2` inside the root) times w2: the norm in front of the next sublayer. One block per row; float32; sums in a
+// fixed order. The new row lies in shared memory (d floats) so that warps can take the sums of the parts whatever their
+// borders: every part is cut into `cuts` slices, a warp sums a slice, a part's slices are added in order.
+constexpr int PAIR_NORM_MAX_SLICES = 1024;
+template <typename TOut>
+__global__ void __launch_bounds__(NORM_THREADS)
+pair_norm_add_kernel(const float* __restrict__ a, const float* __restrict__ wa, float sa, float eps_a,
+                     const float* __restrict__ b, const float* __restrict__ wb, float sb, float eps_b, float* __restrict__ x,
+                     const float* __restrict__ w2, float eps2, int parts, int cuts, TOut* __restrict__ out2, int d,
+                     float* __restrict__ zero, long long zero_count) {
+    extern __shared__ float sum_row[];
+    __shared__ float scratch[32];
+    __shared__ float slice[PAIR_NORM_MAX_SLICES];
+    lp_grid_release();
+    lp_grid_wait();
+    clear_on_the_side(zero, zero_count);
+    const long long row = blockIdx.x;
+    const float* ar = a + row * d;
+    const float* br = b + row * d;
+    float* xr = x + row * d;
+    float s0 = 0.f, s1 = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const float u = ar[i], v = br[i];
+        s0 += u * u;
+        s1 += v * v;
+    }
+    s0 = lp_block_sum(s0, scratch);
+    s1 = lp_block_sum(s1, scratch);
+    const float fa = sa / sqrtf(s0 / (float)d + eps_a), fb = sb / sqrtf(s1 / (float)d + eps_b);
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const float v = xr[i] + (ar[i] * fa * wa[i] + br[i] * fb * wb[i]);
+        xr[i] = v;
+        sum_row[i] = v;
+    }
+    if (!w2) return;
+    __syncthreads();
+    const int width = d / parts, piece = (width + cuts - 1) / cuts;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int k = warp; k < parts * cuts; k += NORM_THREADS / 32) {
+        const int p = k / cuts, lo = (k - p * cuts) * piece, hi = min(width, lo + piece);
+        float ss = 0.f;
+        for (int i = lo + lane; i < hi; i += 32) {
+            const float v = sum_row[p * width + i];
+            ss += v * v;
+        }
+        ss = lp_warp_sum(ss);
+        if (lane == 0) slice[k] = ss;
+    }
+    __syncthreads();
+    TOut* o = out2 + row * d;
+    int held = -1;
+    float f = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const int p = i / width;
+        if (p != held) {
+            float ss = 0.f;
+            for (int c = 0; c < cuts; ++c) ss += slice[p * cuts + c];
+            f = 1.0f / sqrtf(ss / (float)width + eps2);
+            held = p;
+        }
+        o[i] = lp_from_float<TOut>(sum_row[i] * f * w2[i]);
+    }
+}
+
+extern "C" int lp_pair_norm_add(const float* a, const float* wa, float sa, float eps_a, const float* b, const float* wb, float sb,
+                                float eps_b, float* x, const float* w2, float eps2, int parts, void* out2, int out2_dtype, int T,
+                                int d, float* zero, long long zero_count, cudaStream_t stream) {
+    if (T <= 0 || d <= 0) return 0;
+    if (w2 && !out2) LP_REFUSE("pair_norm_add: a following norm without its output");
+    if (parts <= 0 || d % parts || parts > PAIR_NORM_MAX_SLICES) LP_REFUSE("pair_norm_add: rows of %d values in %d equal parts", d, parts);
+    const int cuts = parts >= NORM_THREADS / 32 ? 1 : (NORM_THREADS / 32 + parts - 1) / parts;
+    const size_t smem = (size_t)d * sizeof(float);
+    if (smem > 200 * 1024) LP_REFUSE("pair_norm_add: rows of %d values do not fit shared memory", d);
+#define LP_LAUNCH_PAIR_NORM(TOUT)                                                                                          \
+    do {                                                                                                                   \
+        if (smem > 40 * 1024) {                                                                                            \
+            cudaError_t e = cudaFuncSetAttribute(pair_norm_add_kernel<TOUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) LP_REFUSE("pair_norm_add: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e)); \
+        }                                                                                                                  \
+        lp_launch(pair_norm_add_kernel<TOUT>, T, NORM_THREADS, smem, stream, a, wa, sa, eps_a, b, wb, sb, eps_b, x, w2, eps2, parts, \
+                  cuts, (TOUT*)out2, d, zero, zero_count);                                                                 \
+    } while (0)
+    if (!out2 || out2_dtype == LP_F32) LP_LAUNCH_PAIR_NORM(float);
+    else if (out2_dtype == LP_BF16) LP_LAUNCH_PAIR_NORM(__nv_bfloat16);
+    else LP_REFUSE("pair_norm_add: output dtype code %d", out2_dtype);
+#undef LP_LAUNCH_PAIR_NORM
+    return lp_check_launch("pair_norm_add");
 }

@@ -63,12 +63,26 @@ constexpr int TB = 16;            // tokens per round of loads
 //   chunk's start state where its local state was, and the last one into the sequence's state row)
 //   mode OUTPUT   every chunk starts from its start state and writes its outputs.
 // mode WHOLE is the recurrence in one pass, from and into the sequence's state row (decode steps, short prompts).
-// Variants that other recurrences of this family need: `decay_per_head` (one decay per token and head, decay [T, H], for
-// all its key channels), `key_gain` [T, H] (the key of a token is multiplied by it: an input gate), and `ones` (the last of
+// Variants that other recurrences of this family need: one decay per token and head for all its key channels or one
+// constant per head (`decay_form`), `key_gain` [T, H] (the key of a token is multiplied by it: an input gate), and `ones` (the last of
 // the dv value columns is the constant 1 and the projection holds dv - 1 columns per head: that column of the state is
 // then the decayed sum of the gated keys, and its output their product with the query: a normaliser). `bonus` [H, dk]
 // (the time-mixing family): a token's output is formed from the state BEFORE the token plus u_c k_c v_j for the token
-// itself, o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t, and the state is updated afterwards.
+// itself, o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t, and the state is updated afterwards. `decay_form`: DECAY_CHANNEL
+// (decay [T, H * dk]), DECAY_HEAD (one per token and head, decay [T, H]) or DECAY_FIXED (one constant per head, decay [H]).
+// `angles` [T, rd / 2] (cosine, sine): the first rd channels of queries and keys are rotated as they are loaded, pairs
+// (2i, 2i + 1) or (i, i + rd / 2).
+constexpr int DECAY_CHANNEL = 0, DECAY_HEAD = 1, DECAY_FIXED = 2;
+__device__ __forceinline__ float rotated_channel(const float* head, int c, int rd, int interleaved, const float2* cs) {
+    const float val = head[c];
+    if (c >= rd) return val;
+    const int half = rd >> 1;
+    const bool first = interleaved ? (c & 1) == 0 : c < half;
+    const int pair = interleaved ? c >> 1 : (first ? c : c - half);
+    const float other = head[interleaved ? (c ^ 1) : (first ? c + half : c - half)];
+    const float2 a = cs[pair];
+    return first ? val * a.x - other * a.y : val * a.x + other * a.y;
+}
 constexpr int SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_OUTPUT = 2;
 
 template <int KP, int VT, int KPT, int JT>
@@ -76,9 +90,9 @@ __global__ void __launch_bounds__(VT / JT * KP)
 gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ decay,
                 float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ q_start,
                 float* __restrict__ out, int H, int dk, int dv, float q_scale, int mode, int chunks, int chunk,
-                float* __restrict__ chunk_state, float* __restrict__ chunk_decay, int decay_per_head,
+                float* __restrict__ chunk_state, float* __restrict__ chunk_decay, int decay_form,
                 const float* __restrict__ key_gain, int ones, const float* __restrict__ bonus, int qk_group,
-                const float* __restrict__ beta, int state_cols) {
+                const float* __restrict__ beta, int state_cols, const float2* __restrict__ angles, int rd, int interleaved) {
     extern __shared__ float sm[];
     float* qs = sm;                         // [TB][dk]
     float* ks = qs + TB * dk;
@@ -121,9 +135,13 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
         for (int e = tid; e < nt * dk; e += blockDim.x) {
             const int i = e / dk, c = e - i * dk;
             const float* row = proj + (long long)(tb + i) * ld;
-            qs[e] = row[q_off + (h / qk_group) * dk + c] * q_scale;
-            ks[e] = row[k_off + (h / qk_group) * dk + c] * (key_gain ? key_gain[(long long)(tb + i) * H + h] : 1.0f);
-            as[e] = decay_per_head ? decay[(long long)(tb + i) * H + h] : decay[((long long)(tb + i) * H + h) * dk + c];
+            const float* qh = row + q_off + (h / qk_group) * dk;
+            const float* kh = row + k_off + (h / qk_group) * dk;
+            const float2* cs = angles + (long long)(tb + i) * (rd >> 1);
+            qs[e] = (rd > 0 ? rotated_channel(qh, c, rd, interleaved, cs) : qh[c]) * q_scale;
+            ks[e] = (rd > 0 ? rotated_channel(kh, c, rd, interleaved, cs) : kh[c]) * (key_gain ? key_gain[(long long)(tb + i) * H + h] : 1.0f);
+            as[e] = decay_form == DECAY_FIXED ? decay[h]
+                    : decay_form == DECAY_HEAD ? decay[(long long)(tb + i) * H + h] : decay[((long long)(tb + i) * H + h) * dk + c];
         }
         for (int e = tid; e < nt * VT; e += blockDim.x) {
             const int i = e / VT, c = e - i * VT;
@@ -143,9 +161,11 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
             const float* ki = ks + i * dk;
             const float* ai = as + i * dk;
             if (beta) {
-                // the delta rule (one decay a per head): S <- a S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
-                // Both read-outs are taken from the state before the token, S^T k and S^T q, in one pass of
-                // shuffles: the decayed S^T k is a (S^T k), and o = a (S^T q) + u (k . q).
+                // the delta rule: S <- a S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
+                // Both read-outs are taken from the state before the token's write, S^T k and S^T q, in one pass of
+                // shuffles: o = S^T q + u (k . q) with the decayed S. One decay a per head comes out of the sums (the
+                // decayed S^T k is a (S^T k)); a decay per key channel is applied to the entries first.
+                const bool by_channel = decay_form == DECAY_CHANNEL;
                 float r1[JT], r2[JT], kq = 0.f;
 #pragma unroll
                 for (int jj = 0; jj < JT; ++jj) r1[jj] = r2[jj] = 0.f;
@@ -155,6 +175,11 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
                     if (c < dk) {
                         const float k = ki[c], q = qi[c];
                         kq = fmaf(k, q, kq);
+                        if (by_channel) {
+                            const float ac = ai[c];
+#pragma unroll
+                            for (int jj = 0; jj < JT; ++jj) s[u][jj] *= ac;
+                        }
 #pragma unroll
                         for (int jj = 0; jj < JT; ++jj) {
                             r1[jj] = fmaf(s[u][jj], k, r1[jj]);
@@ -171,7 +196,7 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
                         r2[jj] += __shfl_xor_sync(0xffffffffu, r2[jj], o);
                     }
                 }
-                const float a = ai[0];
+                const float a = by_channel ? 1.0f : ai[0];
                 const float bt = beta[(long long)(tb + i) * H + h];
                 float w[JT];
 #pragma unroll
@@ -453,7 +478,7 @@ token_shift_vec4_kernel(const float* __restrict__ x, float* __restrict__ last, c
 
 // ---------------------------------------------------------------- finish
 // out[t, h * dv + j] = o[t, h, j] / sqrt(mean_j o^2 + eps) * gain[j] * silu(gate[t, h * dv + j]); a warp per (t, h).
-// Variants: rows of o that are `xs` apart (xs > dv: further columns follow a head's values), a gain per head
+// Variants: no gain (null), rows of o that are `xs` apart (xs > dv: further columns follow a head's values), a gain per head
 // (`gain_per_head`: gain [H * dv]), a sigmoid instead of the silu (`gate_sigmoid`), and `max_row` [T, H] (see the kernel).
 template <typename TOut>
 __global__ void __launch_bounds__(256)
@@ -479,9 +504,10 @@ gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ gain, f
     ss = lp_warp_sum(ss);
     const float factor = pre / sqrtf(ss / (float)dv + eps);
     const float* g = gate ? gate + t * ldg + (long long)h * dv : nullptr;
-    const float* gn = gain_per_head ? gain + (long long)h * dv : gain;
+    const float* gn = gain && gain_per_head ? gain + (long long)h * dv : gain;
     for (int j = lane; j < dv; j += 32) {
-        float v = x[j] * factor * gn[j];
+        float v = x[j] * factor;
+        if (gain) v *= gn[j];
         if (g) v *= gate_sigmoid ? 1.0f / (1.0f + expf(-g[j])) : g[j] / (1.0f + expf(-g[j]));
         out[row * dv + j] = lp_from_float<TOut>(v);
     }
@@ -552,6 +578,8 @@ short_conv_kernel(const float* __restrict__ in, int ldi, const TW* __restrict__ 
     }
 }
 
+__device__ __forceinline__ float lp_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
 // ---------------------------------------------------------------- step sizes, decays and write strengths of a recurrence
 // Per token and head, from float32 columns of a projection: dt = softplus(z + dt_bias[h]) (no clamp),
 // decay = exp(-exp(a_log[h]) * dt), and, where a second column zb is given, strength = sigmoid(zb).
@@ -566,10 +594,88 @@ decay_gates_kernel(const float* __restrict__ proj, int ld, int z_off, int b_off,
         const long long t = i / H;
         const int h = (int)(i - t * H);
         const float z = proj[t * ld + z_off + h] + (dt_bias ? dt_bias[h] : 0.f);
-        const float dt = z > 20.f ? z : log1pf(expf(z));
+        const float dt = lp_softplus(z);
         decay[i] = expf(-expf(a_log[h]) * dt);
         if (dt_out) dt_out[i] = dt;
         if (strength) strength[i] = 1.0f / (1.0f + expf(-proj[t * ld + b_off + h]));
+    }
+}
+
+// ---------------------------------------------------------------- gates from low-rank maps
+// Per token, from float32 columns of a projection (the low-rank factors' outputs and the write strengths):
+//   z[c] = sum_r up[c, r] low[r] for the C channels of a map, in float32; then
+//   decays: decay[c] = exp(-exp(a_log[c / dk]) * softplus(z[c] + dt_bias[c]))  (no clamp; one a_log per head of dk channels)
+//   gate:   out[c] = z[c]                                                      (the reader applies its activation)
+//   strength[h] = sigmoid(zb[h])
+// A CTA takes 64 tokens x 64 channels of one of the two maps, 4 x 4 sums per thread; the CTAs of the first column also
+// write their tokens' strengths. grid (column tiles of both maps, token tiles).
+struct RankMap {
+    int off, rank, channels;      // columns [off, off + rank) of the projection -> `channels` outputs
+    const void* up;               // [channels, rank]
+    int up_bf16;
+    float* out;                   // [T, channels]
+};
+constexpr int RM_TILE = 64, RM_K = 32;
+
+__global__ void __launch_bounds__(256)
+low_rank_gates_kernel(const float* __restrict__ proj, int ld, int T, int H, RankMap a, const float* __restrict__ dt_bias,
+                      const float* __restrict__ a_log, int dk, RankMap g, int a_tiles, int b_off, float* __restrict__ strength) {
+    __shared__ float low[RM_TILE][RM_K + 1], up[RM_TILE][RM_K + 1];
+    lp_grid_release();
+    lp_grid_wait();
+    const int t0 = blockIdx.y * RM_TILE;
+    const bool decays = (int)blockIdx.x < a_tiles;
+    const RankMap m = decays ? a : g;
+    const int c0 = (decays ? blockIdx.x : blockIdx.x - a_tiles) * RM_TILE;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int r0 = 0; r0 < m.rank; r0 += RM_K) {
+        for (int e = threadIdx.x; e < RM_TILE * RM_K; e += 256) {
+            const int i = e / RM_K, r = r0 + e % RM_K;
+            const bool in = r < m.rank;
+            low[i][e % RM_K] = (in && t0 + i < T) ? proj[(long long)(t0 + i) * ld + m.off + r] : 0.f;
+            float w = 0.f;
+            if (in && c0 + i < m.channels) {
+                const long long at = (long long)(c0 + i) * m.rank + r;
+                w = m.up_bf16 ? __bfloat162float(((const __nv_bfloat16*)m.up)[at]) : ((const float*)m.up)[at];
+            }
+            up[i][e % RM_K] = w;
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (int r = 0; r < RM_K; ++r) {
+            float x[4], w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { x[i] = low[ty + 16 * i][r]; w[i] = up[tx + 16 * i][r]; }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = t0 + ty + 16 * i;
+        if (t >= T) continue;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int c = c0 + tx + 16 * j;
+            if (c >= m.channels) continue;
+            float v = acc[i][j];
+            if (decays) v = expf(-expf(a_log[c / dk]) * lp_softplus(v + dt_bias[c]));
+            m.out[(long long)t * m.channels + c] = v;
+        }
+    }
+    if (blockIdx.x == 0) {
+        for (int e = threadIdx.x; e < RM_TILE * H; e += 256) {
+            const int t = t0 + e / H, h = e % H;
+            if (t < T) strength[(long long)t * H + h] = 1.0f / (1.0f + expf(-proj[(long long)t * ld + b_off + h]));
+        }
     }
 }
 
@@ -657,8 +763,8 @@ extern "C" int lp_gla_decay(const float* low, int ldl, const void* a2, int w_dty
 extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int v_off, const float* decay, float* state,
                            const int* slots, const int* q_start, float* out, int B, int H, int dk, int dv,
                            float q_scale, int chunks, int chunk, float* chunk_state, float* chunk_decay,
-                           int decay_per_head, const float* key_gain, int ones, const float* bonus, int qk_heads,
-                           const float* beta, cudaStream_t stream) {
+                           int decay_form, const float* key_gain, int ones, const float* bonus, int qk_heads,
+                           const float* beta, const float* angles, int rd, int interleaved, cudaStream_t stream) {
     if (B <= 0) return 0;
     if (chunks < 1) chunks = 1;
     // queries and keys may have fewer heads than the values: head h then reads query / key head h / (H / qk_heads)
@@ -666,7 +772,9 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
     if (H % qk_heads) LP_REFUSE("gla_scan: %d heads over %d query / key heads", H, qk_heads);
     const int qk_group = H / qk_heads;
     const int state_cols = (beta && chunks > 1) ? dv + dk : dv;      // columns of a head in `chunk_state`
-    if (beta && (!decay_per_head || bonus || ones)) LP_REFUSE("gla_scan: the delta rule takes one decay per head and no bonus");
+    if (decay_form < DECAY_CHANNEL || decay_form > DECAY_FIXED) LP_REFUSE("gla_scan: decay form %d", decay_form);
+    if (beta && (bonus || ones)) LP_REFUSE("gla_scan: the delta rule takes no bonus and no constant column");
+    if (rd < 0 || rd > dk || (rd & 1) || (rd > 0 && !angles)) LP_REFUSE("gla_scan: a rotation over %d of %d channels", rd, dk);
     ones = ones ? 1 : 0;
     if (dv - ones <= 0) LP_REFUSE("gla_scan: %d value columns, %d of them constant", dv, ones);
     if (chunks > 1 && (chunk <= 0 || !chunk_state || (!chunk_decay && !beta))) LP_REFUSE("gla_scan: %d chunks without their buffers", chunks);
@@ -686,12 +794,12 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
         if (chunks == 1) {                                                                                            \
             lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_WHOLE, 1, 0, (float*)nullptr,       \
-                      (float*)nullptr, decay_per_head, key_gain, ones, bonus, qk_group, beta, state_cols);                                                                               \
+                      (float*)nullptr, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                               \
         } else {                                                                                                      \
             dim3 grid_local((state_cols + VT_ - 1) / VT_, H, B * chunks);                                             \
             lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid_local, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_LOCAL, chunks, chunk, chunk_state,  \
-                      chunk_decay, decay_per_head, key_gain, ones, bonus, qk_group, beta, state_cols);                                                                                   \
+                      chunk_decay, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                                   \
             const long long per = (long long)H * dv * dk;                                                             \
             if (beta)                                                                                                 \
                 lp_launch(delta_combine_kernel, dim3(dv, H, B), (dk + 31) / 32 * 32, 0, stream, state, slots, q_start, \
@@ -701,7 +809,7 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
                           q_start, chunk_state, (const float*)chunk_decay, H, dk, dv, chunks, chunk);                 \
             lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_OUTPUT, chunks, chunk, chunk_state, \
-                      chunk_decay, decay_per_head, key_gain, ones, bonus, qk_group, beta, state_cols);                                                                                   \
+                      chunk_decay, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                                   \
         }                                                                                                             \
     } while (0)
     // few key channels: 4 threads per column, 64 columns per CTA; from 32 channels on: 16 threads per column, 16 columns
@@ -794,6 +902,28 @@ extern "C" int lp_decay_gates(const float* proj, int ld, int z_off, int b_off, c
     if (blocks > 148 * 8) blocks = 148 * 8;
     lp_launch(decay_gates_kernel, (unsigned)blocks, 256, 0, stream, proj, ld, z_off, b_off, dt_bias, a_log, decay, dt_out, strength, T, H);
     return lp_check_launch("decay_gates");
+}
+
+// proj: float32 [T, ld]; the decays' factor at columns a_off (a_rank), the gate's at g_off (g_rank), H write strengths at
+// b_off. a_up: [H * dk, a_rank], g_up: [g_channels, g_rank] (float32 or bfloat16); dt_bias: float32 [H * dk]; a_log:
+// float32 [H]; decay: float32 [T, H * dk]; gate: float32 [T, g_channels]; strength: float32 [T, H]. g_up null: no gate map.
+extern "C" int lp_low_rank_gates(const float* proj, int ld, int T, int H, int dk, int a_off, int a_rank, const void* a_up,
+                                 int a_dtype, const float* dt_bias, const float* a_log, float* decay, int g_off, int g_rank,
+                                 int g_channels, const void* g_up, int g_dtype, float* gate, int b_off, float* strength,
+                                 cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || dk <= 0 || a_rank <= 0 || a_off < 0 || a_off + a_rank > ld || b_off < 0 || b_off + H > ld)
+        LP_REFUSE("low_rank_gates: %d heads of %d, a factor of %d at %d and strengths at %d of rows of %d", H, dk, a_rank, a_off, b_off, ld);
+    if (g_up && (g_rank <= 0 || g_off < 0 || g_off + g_rank > ld || g_channels <= 0 || !gate)) LP_REFUSE("low_rank_gates: a gate factor of %d at %d of rows of %d", g_rank, g_off, ld);
+    if ((a_dtype != LP_F32 && a_dtype != LP_BF16) || (g_up && g_dtype != LP_F32 && g_dtype != LP_BF16)) LP_REFUSE("low_rank_gates: dtype codes %d and %d", a_dtype, g_dtype);
+    const RankMap a{a_off, a_rank, H * dk, a_up, a_dtype == LP_BF16, decay};
+    const RankMap g{g_off, g_rank, g_up ? g_channels : 0, g_up, g_dtype == LP_BF16, gate};
+    const int a_tiles = (a.channels + RM_TILE - 1) / RM_TILE, g_tiles = (g.channels + RM_TILE - 1) / RM_TILE;
+    const int rows = (T + RM_TILE - 1) / RM_TILE;
+    if (rows > 65535) LP_REFUSE("low_rank_gates: %d tokens exceed the grid", T);
+    lp_launch(low_rank_gates_kernel, dim3(a_tiles + g_tiles, rows), 256, 0, stream, proj, ld, T, H, a, dt_bias, a_log, dk, g, a_tiles,
+              b_off, strength);
+    return lp_check_launch("low_rank_gates");
 }
 
 extern "C" int lp_head_unit_norm(float* x, int ld, int off, int heads, int dim, float eps, float scale, int scaled, int T,

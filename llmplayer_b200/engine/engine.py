@@ -53,9 +53,9 @@ class Engine:
         self._fused = {}               # captured decode steps with upload, argmax and read-back inside
         self._last_ctx: Optional[StepContext] = None
         self._prepared = None          # (context, page tables): the next decode step's pages, reserved ahead
-        from ..cache.sequence_cache import StateRequest
+        from ..cache.sequence_cache import keeps_state
         # whether a run keeps a state that a step changes in place (running a step twice would change it twice)
-        self._keeps_state = any(isinstance(r, StateRequest) or (isinstance(r, tuple) and r) for r in model.cache_requests())
+        self._keeps_state = any(keeps_state(r) for r in model.cache_requests())
 
     # ------------------------------------------------------------------ construction
     @classmethod

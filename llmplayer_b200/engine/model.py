@@ -87,6 +87,7 @@ class Model:
     # ------------------------------------------------------------------ a step
     def forward(self, ctx, cache, rows: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
         """Run the step's tokens through every run and fill ``logits[i]`` for token ``rows[i]``."""
+        ctx.begin_walk()
         d = self.layout.embedding.hidden_size
         x = ctx.buffer("residual", (ctx.num_tokens, d), torch.float32)
         self.embedding.forward(ctx.tokens, x)

@@ -273,6 +273,11 @@ class StepContext:
             cache[key] = table
         return table
 
+    def begin_walk(self) -> None:
+        """The model walk starts (anew, for a context that was moved on): tables formed from the step's positions by an
+        earlier walk are stale, and a walk that is being captured must form its own."""
+        self.__dict__.pop("_angles", None)
+
     def counters(self, name: str, count: int) -> torch.Tensor:
         return self.workspace.get_counters(name, count)
 

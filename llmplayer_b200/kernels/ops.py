@@ -28,12 +28,13 @@ _SIGNATURES = {
         "lp_scaled_sum": [_P, _P, _P, _F, _P, _P, _F, _I, _I, _P],
         "lp_xielu": [_P, _I, _P, _P, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_gated_sum": [_P, _P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P],
-        "lp_rmsnorm": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _P, ctypes.c_longlong, _P],
+        "lp_rmsnorm": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _P, ctypes.c_longlong, _I, _P],
         "lp_rope_cache_write": [_P, _I, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "lp_advance": [_P, _P, _P, _P, _I, _P],
         "lp_rope_angles": [_P, _P, _P, _I, _I, _P],
         "lp_qkv_prepare": [_P, _I, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P,
-                           ctypes.c_longlong, _P, _P, _F, _P],
+                           ctypes.c_longlong, _P, _P, _F, _I, _F, _P],
+        "lp_pair_norm_add": [_P, _P, _F, _F, _P, _P, _F, _F, _P, _P, _F, _I, _P, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_post_norm_add": [_P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P, ctypes.c_longlong, _P, _P, _P],
         "lp_gated_act": [_P, _I, _P, _P, _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_stream_cast": [_P, _P, _I, ctypes.c_longlong, _P, ctypes.c_longlong, _P],
@@ -52,7 +53,7 @@ _SIGNATURES = {
         "lp_gemm_plain": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "attention_plain": {
-        "lp_attention_plain": [_P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _P],
+        "lp_attention_plain": [_P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _P, _P, _P],
     },
     "gemm_tcgen05": {
         "lp_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P,
@@ -63,9 +64,9 @@ _SIGNATURES = {
         "lp_gemm_qkv_rope": [_P, _P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P],
     },
     "attention_mma": {
-        "lp_attention_prefill": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _P],
+        "lp_attention_prefill": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _I, _P, _P, _P],
         "lp_attention_decode": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _P],
-        "lp_attention_decode_fitted": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _P],
+        "lp_attention_decode_fitted": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P],
         "lp_attention_decode_fused": [_P, _I, _P, _I, _I, _P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I,
                                       _I, _I, _I, _P, _F, _I, ctypes.c_longlong, _P, _P],
     },
@@ -87,7 +88,8 @@ _SIGNATURES = {
     },
     "linear_attention": {
         "lp_gla_decay": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _F, _I, _P],
-        "lp_gla_scan": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _I, _P, _I, _P, _I, _P, _P],
+        "lp_gla_scan": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P],
+        "lp_low_rank_gates": [_P, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _P, _I, _P, _P],
         "lp_short_conv": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "lp_decay_gates": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _P],
         "lp_head_unit_norm": [_P, _I, _I, _I, _I, _F, _F, _I, _I, _P],
@@ -392,8 +394,9 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, scale: f
 # --------------------------------------------------------------------------- norm
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
             rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None,
-            clear: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[r] = x[rows[r]] / sqrt(mean(x^2) + eps) * weight, float32 inside.
+            clear: Optional[torch.Tensor] = None, parts: int = 1) -> torch.Tensor:
+    """out[r] = x[rows[r]] / sqrt(mean(x^2) + eps) * weight, float32 inside; ``parts`` > 1: each of that many equal parts
+    of the row is divided by its own root mean square.
 
     ``add`` (same shape as x) is first added into x in place: the residual sum
     fused with the norm that follows it. ``clear``: a float32 buffer that is set to
@@ -423,7 +426,7 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     lib = library("elementwise")
     _check(lib, lib.lp_rmsnorm(x.data_ptr(), _ptr(add), add_code, _ptr(rows), weight.data_ptr(), out.data_ptr(),
                                _code(out, "rmsnorm out"), R, d, float(eps), _ptr(clear),
-                               clear.numel() if clear is not None else 0, _stream()))
+                               clear.numel() if clear is not None else 0, int(parts), _stream()))
     return out
 
 
@@ -882,11 +885,14 @@ def gemm_few(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = ST
 def attention_plain(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, page_table: torch.Tensor,
                     seq_ids: torch.Tensor, positions: torch.Tensor, *, num_heads: int, num_kv_heads: int,
                     head_dim: int, scale: float, window: Optional[int], softcap: Optional[float] = None,
-                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
     """Each query token attends over the cached keys of its sequence up to its own
     position (and within ``window``, if given). ``softcap``: scores become softcap * tanh(score / softcap) after the
     scale; ``sinks``: float32 [H], a logit per head that enters the softmax's denominator once. ``keep_first`` (with a
-    window): the sequence's first ``keep_first`` tokens stay visible to every later query."""
+    window): the sequence's first ``keep_first`` tokens stay visible to every later query. ``chunk`` > 0: a query at
+    position p sees keys of its own chunk only, from p // chunk * chunk on. ``distance`` = (scale, rate), float32 [H] each:
+    the score of a key n positions back loses scale[h] * ln(1 + rate[h] * n)."""
+    dist_scale, dist_rate = _distance_args(distance, num_heads, "attention")
     _check_sinks(sinks, num_heads, "attention")
     _want(q, "attention q", ndim=2)
     _want(out, "attention out", q.dtype, 2)
@@ -905,8 +911,19 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pag
         q.data_ptr(), out.data_ptr(), _code(q, "attention q"), pages.data_ptr(), _code(pages, "attention pages"),
         page_table.data_ptr(), page_table.shape[1], seq_ids.data_ptr(), positions.data_ptr(), T, H, G, hd,
         pages.shape[3], float(scale), int(window) if window else 0, float(softcap or 0.0), _ptr(sinks),
-        int(keep_first) if window else 0, _stream()))
+        int(keep_first) if window else 0, int(chunk or 0), dist_scale, dist_rate, _stream()))
     return out
+
+
+def _distance_args(distance, num_heads: int, what: str):
+    """(pointer, pointer) of a distance bias (scale, rate), or (None, None)."""
+    if distance is None:
+        return None, None
+    for name, t in zip(("scale", "rate"), distance):
+        _want(t, f"{what} distance {name}", torch.float32, 1)
+        if t.numel() != num_heads:
+            raise KernelError(f"{what}: {t.numel()} distance {name}s for {num_heads} heads")
+    return distance[0].data_ptr(), distance[1].data_ptr()
 
 
 def _check_sinks(sinks: Optional[torch.Tensor], num_heads: int, what: str) -> None:
@@ -934,12 +951,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
                       q_start: torch.Tensor, kv_len: torch.Tensor, max_new: int, *, num_heads: int,
                       num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
                       softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-                      exact_weights: bool = False, keep_first: int = 0) -> torch.Tensor:
+                      exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
     """Tensor-core attention for a step that brings several tokens per sequence. ``keep_first`` (with a window): the
     sequence's first ``keep_first`` tokens stay visible to every later query.
     ``q_start`` [B+1]: offsets of each sequence's new tokens; ``kv_len`` [B]: lengths after the step.
     ``exact_weights``: the softmax weights enter the product with the values at float32 precision (as a bfloat16
-    value plus a bfloat16 rest, two products) instead of rounded to bfloat16."""
+    value plus a bfloat16 rest, two products) instead of rounded to bfloat16. ``chunk``, ``distance`` (with
+    ``exact_weights``): see :func:`attention_plain`."""
+    dist_scale, dist_rate = _distance_args(distance, num_heads, "attention_prefill")
     _check_attention(q, out, pages, page_table, num_heads, num_kv_heads, head_dim, "attention_prefill")
     _want(q_start, "attention_prefill q_start", torch.int32, 1)
     _want(kv_len, "attention_prefill kv_len", torch.int32, 1)
@@ -949,7 +968,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
     _check_sinks(sinks, num_heads, "attention_prefill")
     keep_first = int(keep_first) if window else 0
     if (head_dim in (64, 128) and max_new > 64 and tcgen05_attention and not softcap and sinks is None and not exact_weights
-            and not keep_first):
+            and not keep_first and not chunk and distance is None):
         # long runs of new tokens with heads of 64 or 128: scores and P V on the tcgen05 tensor cores
         lib = library("attention_tcgen05")
         _check(lib, lib.lp_attention_prefill_tc(
@@ -963,7 +982,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
         q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1],
         q_start.data_ptr(), kv_len.data_ptr(), B, int(max_new), num_heads, num_kv_heads, head_dim, pages.shape[3],
         float(scale), int(window) if window else 0, float(softcap or 0.0), _ptr(sinks), 1 if exact_weights else 0,
-        keep_first, _stream()))
+        keep_first, int(chunk or 0), dist_scale, dist_rate, _stream()))
     return out
 
 
@@ -993,10 +1012,12 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
                      kv_len: torch.Tensor, scratch, *, num_heads: int, num_kv_heads: int, head_dim: int,
                      scale: float, window: Optional[int], pages_per_split: int = 0, num_splits: int = 0,
                      softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-                     exact_weights: bool = False, keep_first: int = 0) -> torch.Tensor:
+                     exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
     """Tensor-core attention for a step of one token per sequence. ``scratch(name, shape, dtype)``
     supplies the float32 buffer for the partial results of the shares. ``keep_first`` (with a window, shares fitted to
-    the sequences): the sequence's first ``keep_first`` tokens stay visible; their pages are visited first."""
+    the sequences): the sequence's first ``keep_first`` tokens stay visible; their pages are visited first. ``chunk``,
+    ``distance`` (shares fitted to the sequences, ``exact_weights``): see :func:`attention_plain`."""
+    dist_scale, dist_rate = _distance_args(distance, num_heads, "attention_decode")
     _check_attention(q, out, pages, page_table, num_heads, num_kv_heads, head_dim, "attention_decode")
     _want(kv_len, "attention_decode kv_len", torch.int32, 1)
     _check_sinks(sinks, num_heads, "attention_decode")
@@ -1005,8 +1026,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
         raise KernelError(f"attention_decode: {B} sequences, q {tuple(q.shape)}, table {tuple(page_table.shape)}")
     fitted = not pages_per_split or not num_splits
     keep_first = int(keep_first) if window else 0
-    if keep_first and not fitted:
-        raise KernelError("attention_decode: kept first tokens need shares fitted to the sequences")
+    if (keep_first or chunk or distance is not None) and not fitted:
+        raise KernelError("attention_decode: kept first tokens, chunks and distance biases need shares fitted to the sequences")
     if fitted:
         pages_per_split, num_splits = decode_split(B, num_kv_heads, num_heads, page_table.shape[1])
     buf = scratch("attention_partials", (B * num_heads * num_splits * (head_dim + 2),), torch.float32)
@@ -1016,7 +1037,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
             q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1],
             kv_len.data_ptr(), buf.data_ptr(), B, num_heads, num_kv_heads, head_dim, pages.shape[3], float(scale),
             int(window) if window else 0, num_splits, MIN_SHARE_PAGES, float(softcap or 0.0), _ptr(sinks),
-            1 if exact_weights else 0, keep_first, _stream()))
+            1 if exact_weights else 0, keep_first, int(chunk or 0), dist_scale, dist_rate, _stream()))
         return out
     _check(lib, lib.lp_attention_decode(
         q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1], kv_len.data_ptr(),
@@ -1084,24 +1105,25 @@ def attention_decode_fused(qkv: torch.Tensor, rotation: Rotation, out: torch.Ten
 def attention(ctx, q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, page_table: torch.Tensor, *,
               num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
               fast: bool, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-              exact_weights: bool = False, keep_first: int = 0) -> torch.Tensor:
+              exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
     """Attention of the step's tokens over the cache; picks the kernel for the step's shape. ``keep_first`` (with a
-    window): the first tokens of a sequence that stay visible beyond the window."""
+    window): the first tokens of a sequence that stay visible beyond the window. ``chunk``, ``distance``: see
+    :func:`attention_plain`."""
     tensor_cores = (fast and q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16
                     and head_dim % 16 == 0 and head_dim <= 256)
     keep_first = int(keep_first) if window else 0
     if tensor_cores and ctx.all_single:
         return attention_decode(q, out, pages, page_table, ctx.kv_len, ctx.buffer, num_heads=num_heads,
                                 num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale, window=window,
-                                softcap=softcap, sinks=sinks, exact_weights=exact_weights, keep_first=keep_first)
+                                softcap=softcap, sinks=sinks, exact_weights=exact_weights, keep_first=keep_first, chunk=chunk, distance=distance)
     if tensor_cores and not ctx.all_single:
         return attention_prefill(q, out, pages, page_table, ctx.q_start, ctx.kv_len, ctx.max_new,
                                  num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale,
                                  window=window, softcap=softcap, sinks=sinks, exact_weights=exact_weights,
-                                 keep_first=keep_first)
+                                 keep_first=keep_first, chunk=chunk, distance=distance)
     return attention_plain(q, out, pages, page_table, ctx.seq_ids, ctx.positions, num_heads=num_heads,
                            num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale, window=window, softcap=softcap,
-                           sinks=sinks, keep_first=keep_first)
+                           sinks=sinks, keep_first=keep_first, chunk=chunk, distance=distance)
 
 
 # --------------------------------------------------------------------------- latent attention
@@ -1338,7 +1360,8 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
              value_dim: int, q_scale: float, max_new: int = 0, scratch=None, decay_per_head: bool = False,
              key_gain: Optional[torch.Tensor] = None, ones_column: bool = False,
              bonus: Optional[torch.Tensor] = None, qk_heads: Optional[int] = None,
-             delta_strength: Optional[torch.Tensor] = None) -> torch.Tensor:
+             delta_strength: Optional[torch.Tensor] = None, decay_fixed: bool = False, rotation: Optional["Rotation"] = None,
+             angles: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The recurrence S <- diag(decay_t) S + k_t v_t^T, out_t = S^T (q_t * q_scale) over the step's tokens of every
     sequence, from and into ``state`` float32 [slots, H, dv, dk] (row ``slots[b]`` for sequence b; a value column's
     key channels lie together). ``proj``: float32
@@ -1355,11 +1378,13 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     token itself, out_t = (S + diag(bonus) k_t v_t^T)^T q_t, and the state is updated afterwards.
     ``qk_heads``: the projection holds that many query / key heads (a divisor of ``num_heads``); head h reads query / key
     head h // (num_heads // qk_heads). ``delta_strength``: float32 [T, H]; the recurrence is then the gated delta rule
-    (one decay a per head): S <- a S; u = strength * (v - S^T k); S <- S + k u^T; out = S^T q; long prompts run in
+    S <- a S (one decay per head, or one per key channel); u = strength * (v - S^T k); S <- S + k u^T; out = S^T q; long prompts run in
     chunks side by side here too (a chunk's effect on the state that enters it is S -> P S + L with a [dk, dk] matrix P,
-    which the first pass forms beside L)."""
+    which the first pass forms beside L). ``decay_fixed``: ``decay`` is float32 [H], one constant per head. ``rotation``
+    with ``angles`` (float32 [T, rotary_dim / 2, 2], cosines and sines of the step's tokens): queries and keys are rotated
+    as they are read."""
     _want(proj, "gla_scan proj", torch.float32, 2)
-    _want(decay, "gla_scan decay", torch.float32, 2)
+    _want(decay, "gla_scan decay", torch.float32, 1 if decay_fixed else 2)
     _want(state, "gla_scan state", torch.float32, 4)
     _want(slots, "gla_scan slots", torch.int32, 1)
     _want(q_start, "gla_scan q_start", torch.int32, 1)
@@ -1375,15 +1400,22 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
         _want(key_gain, "gla_scan key_gain", torch.float32, 2)
         if key_gain.shape != (T, H):
             raise KernelError(f"gla_scan: key gains {tuple(key_gain.shape)} for {T} tokens and {H} heads")
-    if (decay.shape != (T, H if decay_per_head else H * dk) or state.shape[1:] != (H, dv, dk) or out.shape != (T, H * dv)
+    if (decay.shape != ((H,) if decay_fixed else (T, H if decay_per_head else H * dk)) or state.shape[1:] != (H, dv, dk) or out.shape != (T, H * dv)
             or q_start.numel() != B + 1):
         raise KernelError(f"gla_scan: proj {tuple(proj.shape)}, decay {tuple(decay.shape)}, state {tuple(state.shape)}, "
                           f"out {tuple(out.shape)}, {B} sequences")
     if delta_strength is not None:
         _want(delta_strength, "gla_scan delta_strength", torch.float32, 2)
-        if delta_strength.shape != (T, H) or not decay_per_head:
-            raise KernelError(f"gla_scan: write strengths {tuple(delta_strength.shape)} for {T} tokens and {H} heads "
-                              f"(the delta rule takes one decay per head)")
+        if delta_strength.shape != (T, H):
+            raise KernelError(f"gla_scan: write strengths {tuple(delta_strength.shape)} for {T} tokens and {H} heads")
+    rd = interleaved = 0
+    if rotation is not None and rotation.rotary_dim:
+        _, rd, interleaved = rotation.checked("gla_scan")
+        if angles is None or rd > dk:
+            raise KernelError(f"gla_scan: a rotation over {rd} of {dk} channels needs the tokens' angles")
+        _want(angles, "gla_scan angles", torch.float32, 3)
+        if angles.shape != (T, rd // 2, 2):
+            raise KernelError(f"gla_scan: angles {tuple(angles.shape)} for {T} tokens and {rd} channels")
     if qk_heads is not None and (qk_heads <= 0 or H % qk_heads):
         raise KernelError(f"gla_scan: {H} heads over {qk_heads} query / key heads")
     chunks, chunk_state, chunk_decay = 1, None, None
@@ -1400,22 +1432,24 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     _check(lib, lib.lp_gla_scan(proj.data_ptr(), proj.shape[1], int(q_off), int(k_off), int(v_off), decay.data_ptr(),
                                 state.data_ptr(), slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), B, H, dk, dv,
                                 float(q_scale), chunks, chunk, _ptr(chunk_state), _ptr(chunk_decay),
-                                1 if decay_per_head else 0, _ptr(key_gain), 1 if ones_column else 0, _ptr(bonus),
-                                int(qk_heads or H), _ptr(delta_strength), _stream()))
+                                2 if decay_fixed else 1 if decay_per_head else 0, _ptr(key_gain), 1 if ones_column else 0,
+                                _ptr(bonus), int(qk_heads or H), _ptr(delta_strength), _ptr(angles) if rd else None, rd,
+                                interleaved, _stream()))
     if chunks > 1:
         count_launches(2)
     return out
 
 
-def gla_finish(o: torch.Tensor, gain: torch.Tensor, eps: float, gate: Optional[torch.Tensor], out: torch.Tensor, *,
+def gla_finish(o: torch.Tensor, gain: Optional[torch.Tensor], eps: float, gate: Optional[torch.Tensor], out: torch.Tensor, *,
                num_heads: int, value_dim: int, clear: Optional[torch.Tensor] = None, gain_per_head: bool = False,
                gate_sigmoid: bool = False, max_row: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t, h] = rmsnorm(o[t, h]) * gain * silu(gate[t, h]) per head of ``value_dim`` values; ``gate``: float32
-    [T, H * dv] (may be a column slice) or None. ``gain_per_head``: ``gain`` is [H * dv]. ``gate_sigmoid``: the gate's
+    [T, H * dv] (may be a column slice) or None. ``gain`` None: no gain. ``gain_per_head``: ``gain`` is [H * dv]. ``gate_sigmoid``: the gate's
     sigmoid instead of its silu. ``max_row`` (float32 [T, H]): ``o`` is [T, H * (dv + 1)], a head's last column being
     its normaliser n; o[t, h] is first divided by max(|n|, exp(-max_row[t, h])) + 1e-6."""
     _want(o, "gla_finish o", torch.float32, 2)
-    _want(gain, "gla_finish gain", torch.float32, 1)
+    if gain is not None:
+        _want(gain, "gla_finish gain", torch.float32, 1)
     _want(out, "gla_finish out", ndim=2)
     T = o.shape[0]
     xs = value_dim + (1 if max_row is not None else 0)
@@ -1424,15 +1458,15 @@ def gla_finish(o: torch.Tensor, gain: torch.Tensor, eps: float, gate: Optional[t
         if max_row.shape != (T, num_heads):
             raise KernelError(f"gla_finish: maxima {tuple(max_row.shape)} for {T} tokens and {num_heads} heads")
     if (o.shape != (T, num_heads * xs) or out.shape != (T, num_heads * value_dim)
-            or gain.numel() != (num_heads * value_dim if gain_per_head else value_dim)):
-        raise KernelError(f"gla_finish: o {tuple(o.shape)}, out {tuple(out.shape)}, gain {tuple(gain.shape)}")
+            or (gain is not None and gain.numel() != (num_heads * value_dim if gain_per_head else value_dim))):
+        raise KernelError(f"gla_finish: o {tuple(o.shape)}, out {tuple(out.shape)}, gain {None if gain is None else tuple(gain.shape)}")
     gp, ldg = (None, 0)
     if gate is not None:
         gp, ldg = _slice(gate, "gla_finish gate")
         if gate.shape != out.shape:
             raise KernelError(f"gla_finish: gate {tuple(gate.shape)} does not match out {tuple(out.shape)}")
     lib = library("linear_attention")
-    _check(lib, lib.lp_gla_finish(o.data_ptr(), gain.data_ptr(), float(eps), gp, ldg, out.data_ptr(),
+    _check(lib, lib.lp_gla_finish(o.data_ptr(), _ptr(gain), float(eps), gp, ldg, out.data_ptr(),
                                   _code(out, "gla_finish out"), T, num_heads, value_dim, *_clear_args(clear, "gla_finish"),
                                   xs, 1 if gain_per_head else 0, 1 if gate_sigmoid else 0, _ptr(max_row), _stream()))
     return out
@@ -1490,6 +1524,38 @@ def decay_gates(proj: torch.Tensor, z_off: int, dt_bias: Optional[torch.Tensor],
     lib = library("linear_attention")
     _check(lib, lib.lp_decay_gates(proj.data_ptr(), proj.shape[1], int(z_off), int(b_off), _ptr(dt_bias), a_log.data_ptr(),
                                    decay.data_ptr(), _ptr(dt), _ptr(strength), T, H, _stream()))
+
+
+def low_rank_gates(proj: torch.Tensor, a_off: int, a_up: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                   decay: torch.Tensor, b_off: int, strength: torch.Tensor, *, key_dim: int, g_off: int = 0,
+                   g_up: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """Gates of a recurrence from low-rank maps, per token, all in float32: decay[t, c] = exp(-exp(a_log[c // key_dim]) *
+    softplus(a_up[c] . proj[t, a_off:a_off + rank] + dt_bias[c])), strength[t, h] = sigmoid(proj[t, b_off + h]) and, with
+    ``g_up``, gate[t, c] = g_up[c] . proj[t, g_off:g_off + rank] (before any activation). ``proj``: float32 [T, F];
+    ``a_up``: [H * key_dim, rank]; ``decay``: float32 [T, H * key_dim]; ``strength``: float32 [T, H]."""
+    _want(proj, "low_rank_gates proj", torch.float32, 2)
+    _want(a_up, "low_rank_gates a_up", ndim=2)
+    _want(dt_bias, "low_rank_gates dt_bias", torch.float32, 1)
+    _want(a_log, "low_rank_gates a_log", torch.float32, 1)
+    _want(decay, "low_rank_gates decay", torch.float32, 2)
+    _want(strength, "low_rank_gates strength", torch.float32, 2)
+    T, H = strength.shape
+    C = H * key_dim
+    if proj.shape[0] != T or decay.shape != (T, C) or a_up.shape[0] != C or dt_bias.numel() != C or a_log.numel() != H:
+        raise KernelError(f"low_rank_gates: proj {tuple(proj.shape)}, a_up {tuple(a_up.shape)}, decay {tuple(decay.shape)}, {H} heads of {key_dim}")
+    rank_g = channels = code = 0
+    if g_up is not None:
+        _want(g_up, "low_rank_gates g_up", ndim=2)
+        _want(gate, "low_rank_gates gate", torch.float32, 2)
+        channels, rank_g = g_up.shape
+        code = _code(g_up, "low_rank_gates g_up")
+        if gate.shape != (T, channels):
+            raise KernelError(f"low_rank_gates: g_up {tuple(g_up.shape)}, gate {tuple(gate.shape)}")
+    lib = library("linear_attention")
+    _check(lib, lib.lp_low_rank_gates(
+        proj.data_ptr(), proj.shape[1], T, H, int(key_dim), int(a_off), a_up.shape[1], a_up.data_ptr(), _code(a_up, "low_rank_gates a_up"),
+        dt_bias.data_ptr(), a_log.data_ptr(), decay.data_ptr(), int(g_off), rank_g, channels, _ptr(g_up), code, _ptr(gate),
+        int(b_off), strength.data_ptr(), _stream()))
 
 
 def head_unit_norm(x: torch.Tensor, offset: int, heads: int, dim: int, eps: float, scale: float = 1.0,
@@ -1590,15 +1656,17 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
                 seq_ids: torch.Tensor, page_table: torch.Tensor, q_out: torch.Tensor, pages: torch.Tensor, *,
                 num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, unit_norm_eps: Optional[float],
                 clear: Optional[torch.Tensor] = None, q_gain: Optional[torch.Tensor] = None,
-                k_gain: Optional[torch.Tensor] = None, gain_eps: float = 0.0, write_kv: bool = True) -> None:
+                k_gain: Optional[torch.Tensor] = None, gain_eps: float = 0.0, write_kv: bool = True,
+                value_norm_eps: Optional[float] = None) -> None:
     """From the float32 projection ``qkv`` [T, H * dk + G * dk + G * dv]: add ``bias`` (float32, same width, or None),
     rotate queries and keys, divide each query and key head by its root mean square (``unit_norm_eps`` not None), and
     store queries to ``q_out`` [T, H * hdp] and keys and values into ``pages`` [num_pages, 2, G, page_size, hdp], every
     head padded with zeros to the pages' head size hdp. ``q_gain`` / ``k_gain`` (float32 [dk], shared by the heads):
     before the rotation, query / key heads are RMS-normed over dk with that gain and ``gain_eps``. ``write_kv=False``:
     ``qkv`` [T, H * dk] holds queries only (a layer that attends over another layer's keys and values); ``pages`` only
-    says how queries are stored."""
-    _want(qkv, "qkv_prepare qkv", torch.float32, 2)
+    says how queries are stored. ``value_norm_eps``: every value head is divided by its root mean square over dv before it
+    is stored. ``qkv`` may be a column slice of a wider product."""
+    qkv_ptr, qkv_ld = _slice(qkv, "qkv_prepare qkv")
     _want(positions, "qkv_prepare positions", torch.int32, 1)
     _want(seq_ids, "qkv_prepare seq_ids", torch.int32, 1)
     _want(page_table, "qkv_prepare page_table", torch.int32, 2)
@@ -1626,11 +1694,12 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
     freq_ptr, rotary_dim, interleaved = rotation.checked("qkv_prepare")
     lib = library("elementwise")
     _check(lib, lib.lp_qkv_prepare(
-        qkv.data_ptr(), qkv.shape[1], _ptr(bias), freq_ptr, positions.data_ptr(), seq_ids.data_ptr(),
+        qkv_ptr, qkv_ld, _ptr(bias), freq_ptr, positions.data_ptr(), seq_ids.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], q_out.data_ptr(), _code(q_out, "qkv_prepare q_out"),
         pages.data_ptr() if write_kv else None, _code(pages, "qkv_prepare pages"), T, H, G, dk, dv, hdp, rotary_dim, interleaved,
         0 if unit_norm_eps is None else 1, float(unit_norm_eps or 0.0), pages.shape[3], *_clear_args(clear, "qkv_prepare"),
-        _ptr(q_gain), _ptr(k_gain) if write_kv else None, float(gain_eps), _stream()))
+        _ptr(q_gain), _ptr(k_gain) if write_kv else None, float(gain_eps), 0 if value_norm_eps is None else 1,
+        float(value_norm_eps or 0.0), _stream()))
 
 
 def post_norm_add(y: torch.Tensor, weight: torch.Tensor, eps: float, x: torch.Tensor, *, next_weight: Optional[torch.Tensor] = None,
@@ -1665,6 +1734,37 @@ def post_norm_add(y: torch.Tensor, weight: torch.Tensor, eps: float, x: torch.Te
     _check(lib, lib.lp_post_norm_add(y.data_ptr(), weight.data_ptr(), float(eps), x.data_ptr(), _ptr(next_weight),
                                      float(next_eps), _ptr(next_out), code, T, d,
                                      *_clear_args(clear, "post_norm_add"), _ptr(y_bias), _ptr(scale), _stream()))
+    return x
+
+
+def pair_norm_add(a: torch.Tensor, a_weight: torch.Tensor, a_scale: float, a_eps: float, b: torch.Tensor, b_weight: torch.Tensor,
+                  b_scale: float, b_eps: float, x: torch.Tensor, *, next_weight: Optional[torch.Tensor] = None,
+                  next_eps: float = 0.0, next_parts: int = 1, next_out: Optional[torch.Tensor] = None,
+                  clear: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += a_scale * rmsnorm(a, a_weight) + b_scale * rmsnorm(b, b_weight), float32 [T, d] in place; with ``next_weight``,
+    also next_out = the RMS norm of the new x in ``next_parts`` equal parts (each divided by its own root mean square),
+    times ``next_weight``: the norm in front of the next sublayer. ``clear``: a float32 buffer zeroed on the side."""
+    for name, t in (("a", a), ("b", b), ("x", x)):
+        _want(t, f"pair_norm_add {name}", torch.float32, 2)
+        if t.shape != x.shape:
+            raise KernelError(f"pair_norm_add: {name} {tuple(t.shape)} does not match x {tuple(x.shape)}")
+    T, d = x.shape
+    for name, t in (("a_weight", a_weight), ("b_weight", b_weight), ("next_weight", next_weight)):
+        if t is not None:
+            _want(t, f"pair_norm_add {name}", torch.float32, 1)
+            if t.numel() != d:
+                raise KernelError(f"pair_norm_add: {name} of {t.numel()} values for rows of {d}")
+    code = F32
+    if next_weight is not None:
+        _want(next_out, "pair_norm_add next_out", ndim=2)
+        if next_out.shape != x.shape:
+            raise KernelError(f"pair_norm_add: next output {tuple(next_out.shape)} for x {tuple(x.shape)}")
+        code = _code(next_out, "pair_norm_add next_out")
+    lib = library("elementwise")
+    _check(lib, lib.lp_pair_norm_add(a.data_ptr(), a_weight.data_ptr(), float(a_scale), float(a_eps), b.data_ptr(), b_weight.data_ptr(),
+                                     float(b_scale), float(b_eps), x.data_ptr(), _ptr(next_weight), float(next_eps), int(next_parts),
+                                     _ptr(next_out) if next_weight is not None else None, code, T, d,
+                                     *_clear_args(clear, "pair_norm_add"), _stream()))
     return x
 
 

@@ -44,6 +44,12 @@ class Attention(Part):
             raise ConfigError("a layer that attends over another layer's keys and values keeps no first tokens of its own")
         if s.softcap is not None and not s.softcap > 0:
             raise ConfigError(f"score cap must be positive or absent, got {s.softcap}")
+        if s.chunk is not None and (s.chunk <= 0 or s.keep_first or s.shares_kv):
+            raise ConfigError(f"chunks of {s.chunk} positions: they must be positive and go with neither kept first tokens nor shared keys")
+        if (s.distance_scale is None) != (s.distance_rate is None) or (s.distance_scale is not None and not s.exact_weights):
+            raise ConfigError("a distance bias has a scale and a rate per head and comes with softmax weights at float32 precision")
+        if s.value_norm_eps is not None and (s.shares_kv or not s.value_norm_eps > 0):
+            raise ConfigError("normed values need keys and values of the layer's own and a positive constant")
         self.spec = spec
         self.position = POSITIONS.build(s.position)
         self.qkv: Optional[Linear] = None
@@ -56,6 +62,9 @@ class Attention(Part):
         self.q_gain: Optional[torch.Tensor] = None
         self.k_gain: Optional[torch.Tensor] = None
         self.output_bias: Optional[torch.Tensor] = None     # float32 [hidden]: what the output projection adds
+        self.distance = None                                # (scale, rate), float32 [heads] each
+        self.inputs_stacked = False                         # set by an owner whose one product covers this part's inputs
+        self._inputs = []
 
     @property
     def capture_safe(self) -> bool:
@@ -83,13 +92,19 @@ class Attention(Part):
                 specs[name] = TensorSpec((s.head_dim,), GAIN)
         if s.o_bias is not None:
             specs[s.o_bias] = TensorSpec((s.hidden_size,), BIAS)
+        for name in (s.distance_scale, s.distance_rate):
+            if name is not None:
+                specs[name] = TensorSpec((s.num_heads,), BIAS)
         return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         super().load(tensors, runtime)
         s = self.spec
         names = [s.q] if s.shares_kv else [s.q, s.k, s.v]
-        self.qkv = Linear([tensors[n] for n in names], runtime)      # rows: queries, keys, values
+        self._inputs = [tensors[n] for n in names]                   # rows: queries, keys, values
+        if not self.inputs_stacked:
+            self.qkv = Linear(self._inputs, runtime)
+            self._inputs = []
         o = tensors[s.o]
         if self.stored_dim != self.value_dim:
             # the attention kernels leave heads of stored_dim values (zeros beyond value_dim): give `o` columns to match
@@ -111,6 +126,8 @@ class Attention(Part):
         self.q_gain = runtime.gain(tensors[s.q_norm]) if s.q_norm is not None else None
         self.k_gain = runtime.gain(tensors[s.k_norm]) if s.k_norm is not None else None
         self.output_bias = runtime.gain(tensors[s.o_bias]) if s.o_bias is not None else None
+        if s.distance_scale is not None:
+            self.distance = (runtime.gain(tensors[s.distance_scale]), runtime.gain(tensors[s.distance_rate]))
 
     # ------------------------------------------------------------------ cache
     def cache_request(self):
@@ -118,9 +135,19 @@ class Attention(Part):
         if s.shares_kv:
             return None
         return KVRequest(s.num_kv_heads, self.stored_dim, s.window if s.cache_window == "own" else s.cache_window,
-                         int(s.keep_first or 0))
+                         int(s.keep_first or 0), s.chunk)
 
     # ------------------------------------------------------------------ step
+    @property
+    def offers_inputs(self) -> bool:
+        """Whether an owner may form this part's input projections in a wider product (the general path only)."""
+        return self.spec.general
+
+    def take_inputs(self):
+        """The matrices that multiply the part's input, for an owner that set ``inputs_stacked`` before the load."""
+        taken, self._inputs = self._inputs, []
+        return taken
+
     def buffer_to_clear(self, ctx, tokens: int):
         return self.qkv.sums_into(ctx, tokens, "qkv", ops.STORE)
 
@@ -151,22 +178,30 @@ class Attention(Part):
 
     def _forward_general(self, ctx, cache, x, residual: torch.Tensor, then_norm=None, overwrite: bool = False,
                          bias_later: bool = False) -> bool:
-        """A layer with biases, normed heads, capped scores, sinks or values of another size than its keys:
+        """A layer with biases, normed heads, capped scores, sinks, chunks, distance biases or values of another size than its keys:
         projection with float32 sums, one kernel that adds the biases, norms, rotates and stores queries, keys and
         values (heads padded to ``stored_dim``), then the attention kernels with the cap and the sinks as arguments.
         A layer that attends over another run's keys and values projects and prepares queries only."""
-        s, rt = self.spec, self.runtime
         if isinstance(x, PendingNorm):
             x = x.tensor()
-        T = x.shape[0]
+        qkv = ctx.buffer("qkv", (x.shape[0], self.qkv.out_features), torch.float32)
+        with ops.section("attention.qkv"):
+            self.qkv.store(x, qkv, ctx)
+        return self.forward_projected(ctx, cache, qkv, 0, residual, then_norm=then_norm, overwrite=overwrite, bias_later=bias_later)
+
+    def forward_projected(self, ctx, cache, proj: torch.Tensor, offset: int, residual: torch.Tensor, then_norm=None,
+                          overwrite: bool = True, bias_later: bool = False) -> bool:
+        """The general path from the input projections on: ``proj`` float32 [T, F] holds queries, keys and values from
+        column ``offset``. Stores the layer's output in ``residual`` (``overwrite``) or adds it there."""
+        s, rt = self.spec, self.runtime
+        T = proj.shape[0]
         H, G, hd = s.num_heads, s.num_kv_heads, self.stored_dim
         rotation = self.position.rotation()
         if rotation is None:
             raise ConfigError("the general attention path applies rotations only (a position part with rotation())")
         table = ctx.page_tables[cache.group_index]
-        qkv = ctx.buffer("qkv", (T, self.qkv.out_features), torch.float32)
-        with ops.section("attention.qkv"):
-            self.qkv.store(x, qkv, ctx)
+        width = H * s.head_dim + (0 if s.shares_kv else G * (s.head_dim + self.value_dim))
+        qkv = proj if offset == 0 and proj.shape[1] == width else proj[:, offset:offset + width]
         q = ctx.buffer("q", (T, H * hd), rt.act_dtype)
         with ops.section("attention.position"):
             # an output product that sums partial results wants its target zero: this kernel clears it on the side
@@ -174,12 +209,12 @@ class Attention(Part):
             ops.qkv_prepare(qkv, self.bias, rotation, ctx.positions, ctx.seq_ids, table, q, cache.pages, num_heads=H,
                             num_kv_heads=G, key_dim=s.head_dim, value_dim=self.value_dim, unit_norm_eps=s.unit_norm_eps,
                             clear=clear, q_gain=self.q_gain, k_gain=self.k_gain, gain_eps=s.qk_norm_eps,
-                            write_kv=not s.shares_kv)
+                            write_kv=not s.shares_kv, value_norm_eps=s.value_norm_eps)
         o = ctx.buffer("attn_out", (T, H * hd), rt.act_dtype)
         with ops.section("attention.scores"):
             ops.attention(ctx, q, o, cache.pages, table, num_heads=H, num_kv_heads=G, head_dim=hd, scale=s.scale,
                           window=s.window, fast=rt.fast, softcap=s.softcap, sinks=self.sinks, exact_weights=s.exact_weights,
-                          keep_first=int(s.keep_first or 0))
+                          keep_first=int(s.keep_first or 0), chunk=int(s.chunk or 0), distance=self.distance)
         with ops.section("attention.out"):
             if overwrite:
                 if clear is not None:

@@ -73,7 +73,7 @@ class PreNormBlock(Part):
 
         # a part that takes a pending norm gets (stream, norm) and may apply the norm in its first product
         mixer_pends = bool(getattr(self.mixer, "takes_pending_norm", False))
-        ffn_pends = bool(getattr(self.ffn, "takes_pending_norm", False))
+        ffn_pends = bool(getattr(self.ffn, "takes_pending_norm", False)) and bool(getattr(self.ffn_norm, "fusable_rms", False))
         if normed_ready:
             mixer_in = h
         elif mixer_pends:
@@ -181,9 +181,10 @@ class ParallelBlock(Part):
             part.load(tensors, runtime)
         stacked, at = [], 0
         self._mixer_at = self._mixer_gate_at = self._ffn_gate_at = self._up_at = None
-        if hasattr(self.mixer, "input_projections"):
+        offered = self.mixer.input_projections() if hasattr(self.mixer, "input_projections") else None
+        if offered:
             self._mixer_at = at
-            for m in self.mixer.input_projections():
+            for m in offered:
                 stacked.append(m)
                 at += m.shape[0]
         self.mixer_gate_bias = self.ffn_gate_bias = None

@@ -1,5 +1,5 @@
-"""Norms of the residual stream, in float32: RMS norm, out = x / sqrt(mean(x^2) + eps) * gain, and
-layer norm with a gain and no bias.
+"""Norms of the residual stream, in float32: RMS norm, out = x / sqrt(mean(x^2) + eps) * gain, over whole rows or over
+equal parts of a row (each with its own root mean square), and layer norm with a gain and no bias.
 
 Reference: inference/RMSNorm.java:17-35, tensor/ScalarOps.java:26-35,
 src/main/resources/kernels/cuda/rmsnorm.cu:6-46. The gain is used as stored.
@@ -18,10 +18,14 @@ from .specs import GAIN, NormSpec, TensorSpec
 
 class RMSNorm(Part):
     capture_safe = True
-    fusable_rms = True      # a product that adds into the residual stream may write this norm on the way
 
     def __init__(self, spec: NormSpec):
+        if spec.groups <= 0 or spec.size % spec.groups:
+            raise ConfigError(f"a row of {spec.size} values cannot be normed in {spec.groups} equal parts")
         self.spec = spec
+        self.rms_parts = spec.groups            # a kernel that norms the stream in so many equal parts may write this norm
+        # a product that adds into the residual stream, or reads it, may apply this norm on the way (one factor per row)
+        self.fusable_rms = spec.groups == 1
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
@@ -35,7 +39,7 @@ class RMSNorm(Part):
               add: Optional[torch.Tensor] = None, clear: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``out[r] = norm(x[rows[r]])``; ``add`` is summed into ``x`` first (in place);
         ``clear`` is a float32 buffer zeroed on the side."""
-        return ops.rmsnorm(x, self.weight, self.spec.eps, out, rows=rows, add=add, clear=clear)
+        return ops.rmsnorm(x, self.weight, self.spec.eps, out, rows=rows, add=add, clear=clear, parts=self.rms_parts)
 
 
 class LayerNorm(Part):

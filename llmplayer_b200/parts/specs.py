@@ -44,11 +44,13 @@ class TensorSpec:
 @dataclass(frozen=True)
 class NormSpec:
     """``kind="rmsnorm"``: x / sqrt(mean(x^2) + eps) * weight. ``kind="layernorm"``: (x - mean) /
-    sqrt(variance + eps) * weight, the variance being the mean squared deviation; no bias."""
+    sqrt(variance + eps) * weight, the variance being the mean squared deviation; no bias. ``groups`` > 1 (RMS norm):
+    the row is cut into that many equal parts, each divided by its own root mean square; the weight spans the row."""
     size: int
     eps: float
     weight: str
     kind: str = "rmsnorm"
+    groups: int = 1
 
 
 @dataclass(frozen=True)
@@ -128,12 +130,18 @@ class AttentionSpec:
     # further back than the layer itself; "own": the layer's own ``window``.
     cache_window: object = "own"
     keep_first: Optional[int] = None     # with ``window``: a sequence's first so many tokens stay visible to every later query, at their true positions
+    chunk: Optional[int] = None          # a query at position p sees keys j <= p of its own chunk only: j // chunk == p // chunk
+    # the score of a key at distance n loses distance_scale[h] * ln(1 + distance_rate[h] * n) (tensors [heads], both or neither)
+    distance_scale: Optional[str] = None
+    distance_rate: Optional[str] = None
+    value_norm_eps: Optional[float] = None   # every value head is divided by its root mean square (no gain) and cached so
 
     @property
     def general(self) -> bool:
         return (bool(self.keep_first) or self.value_dim not in (None, self.head_dim) or any(b is not None for b in (self.q_bias, self.k_bias, self.v_bias))
                 or self.unit_norm_eps is not None or self.softcap is not None or self.sink is not None or self.exact_weights
-                or self.q_norm is not None or self.k_norm is not None or self.o_bias is not None or self.sink_value is not None)
+                or self.q_norm is not None or self.k_norm is not None or self.o_bias is not None or self.sink_value is not None
+                or self.chunk is not None or self.distance_scale is not None or self.value_norm_eps is not None)
 
 
 @dataclass(frozen=True)
@@ -279,7 +287,13 @@ class GatedDeltaRuleSpec:
     Per head: strength = sigmoid(``strength`` x), decay = exp(-exp(``a_log``) softplus(``decay`` x + ``dt_bias``));
     S <- decay S; u = strength (v - S^T k); S <- S + k u^T; o = S^T q. Each head's o is divided by its root mean square
     over value_dim (``norm_eps``), times ``out_norm`` [value_dim] (shared by the heads), times silu(``gate`` x); then ``o``.
-    The state and the convolutions' last inputs are float32 and start at zero."""
+    The state and the convolutions' last inputs are float32 and start at zero.
+
+    ``decay_up``: one decay per head AND key channel from a low-rank map: the pre-activations are ``decay_up`` (``decay`` x)
+    with ``decay`` [rank, hidden], ``decay_up`` [num_heads * key_dim, rank] and ``dt_bias`` [num_heads * key_dim] (``a_log``
+    stays one number per head); S <- diag(decay) S then decays every key channel's row by its own factor. ``gate_up``:
+    the output gate's pre-activations are ``gate_up`` (``gate`` x) with ``gate`` [rank, hidden]. The ranks are read off the
+    file. ``gate_activation``: "silu" or "sigmoid"."""
     hidden_size: int
     num_heads: int
     num_qk_heads: int
@@ -301,17 +315,45 @@ class GatedDeltaRuleSpec:
     out_norm: str
     o: str
     kind: str = "gated_delta_rule"
+    decay_up: Optional[str] = None
+    gate_up: Optional[str] = None
+    gate_activation: str = "silu"
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with a fixed decay per head and neither softmax nor denominator (retention). q = ``q`` x and k =
+    ``k`` x have ``num_heads`` heads of ``key_dim``, v = ``v`` x heads of ``value_dim``; ``position`` rotates q and k, k is
+    multiplied by key_dim^-1/2. Per head: S_t = ``decays``[h] S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (float32, S zero at a
+    sequence's start). Each head's o is divided by its root mean square over value_dim (``norm_eps``, no gain), the heads
+    are multiplied by silu(``gate`` x) and projected by ``o``."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    norm_eps: float
+    position: PositionSpec
+    decays: Tuple[float, ...]
+    q: str
+    k: str
+    v: str
+    gate: str
+    o: str
+    kind: str = "retention"
 
 
 @dataclass(frozen=True)
 class MixerPairSpec:
     """Two mixers side by side that read the same input: ``left_scale`` * left(x) + ``right_scale`` * right(x). Each
-    keeps its own cache or state."""
+    keeps its own cache or state. ``left_norm`` / ``right_norm`` (both or neither): each result is RMS-normed over the
+    width before it is scaled and summed."""
     left: object
     right: object
     left_scale: float = 1.0
     right_scale: float = 1.0
     kind: str = "mixer_pair"
+    left_norm: Optional[NormSpec] = None
+    right_norm: Optional[NormSpec] = None
 
 
 @dataclass(frozen=True)
