@@ -6,6 +6,7 @@
     python bench.py --design botuvik [--size s|m|l] [--layers N]      (the same for the Botuvik design, beside both)
     python bench.py --design zasitar [--size s|m|l] [--layers N]      (the Zasitar design beside Botuvik and Llama)
     python bench.py --design dopuvik [--size s|m|l] [--layers N]      (the Dopuvik design beside Zasitar and Llama)
+    python bench.py --design vomotar [--size s|m|l] [--layers N]      (the Vomotar design beside Dopuvik and Llama)
 
 One "step" is one decode step of the whole batch. The default run has the Llama-3.2-1B shape, a batch of 8
 sequences with 512-token prompts in a cache sized for a context of 4096. Every figure comes from the library's
@@ -32,6 +33,9 @@ and routed feed-forwards) beside Ramupel, the closest existing design (a recurre
 ``--design dopuvik`` does the same for the Dopuvik design (state-space layers, latent attention in a window, attention
 with kept first tokens beside a gated delta rule, experts chosen in groups with identity experts) beside Zasitar, the
 closest existing design (a recurrence among windowed attention layers, routed experts), and Llama.
+``--design vomotar`` does the same for the Vomotar design (a delta rule with a decay per key channel, attention in chunks
+with a distance bias beside a retention, dense feed-forwards) beside Dopuvik, the closest existing design (delta rule,
+attention beside a recurrence), and Llama.
 ``--design zasitar`` does the same for the Zasitar design (time-mixing layers, sliding-window attention with normed
 heads and keys shared between layers, results normed behind the sublayers) beside Botuvik, the closest existing design
 (a matrix recurrence among attention layers with sinks, dense and routed feed-forwards), and Llama.
@@ -253,6 +257,27 @@ def dopuvik_config(size, layers):
             "logit_scale": 1.0, "layers": [dict(order[i % 4], mlp=routed) for i in range(layers)]}
 
 
+VOMOTAR_CHUNK = 1024           # half of the measured prompt, as long as the window of the Dopuvik beside it
+
+
+def vomotar_config(size, layers):
+    """Of every four layers the first is attention (grouped as in the Llama beside it, in chunks of VOMOTAR_CHUNK tokens)
+    beside a retention (the heads of the Ramupel design's linear attention, rotated), the other three a delta rule with a
+    decay per key channel (the heads of the Dopuvik design's delta rule, convolutions of 4 taps, low-rank maps of the head
+    size). Norms in two parts; dense feed-forwards of the Llama's size."""
+    width, heads, _, (gh, gk, gv), ff = HYBRID_SIZES[size]
+    hd = width // heads
+    pair = {"type": "parallel",
+            "mixer": {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+                               "mask": {"size": VOMOTAR_CHUNK}},
+                      "right": {"heads": gh, "dim": gk, "vdim": gv, "decay": [1.0 - 2.0 ** (-5 - i % 8) for i in range(gh)],
+                                "rot": {"base": 10000.0, "dims": gk}}}}
+    delta = {"type": "channel_delta", "mixer": {"heads": gh, "kv_heads": gh, "dim": gk, "vdim": gk, "conv": 4}}
+    dense = {"kind": "dense", "ff": (2 * ff // 3 + 127) // 128 * 128}
+    return {"architecture": "Vomotar", "vocab": 32000, "width": width, "norm": {"eps": 1e-5, "groups": 2},
+            "layers": [dict(delta if i % 4 else pair, mlp=dense) for i in range(layers)]}
+
+
 def compare_designs(args, peaks) -> int:
     import torch
     from llmplayer_b200 import Engine
@@ -269,8 +294,10 @@ def compare_designs(args, peaks) -> int:
     clocks = ClockSampler()
     clocks.start()
     botuvik, zasitar, dopuvik = args.design == "botuvik", args.design == "zasitar", args.design == "dopuvik"
+    vomotar = args.design == "vomotar"
     title = {"botuvik": "Botuvik design beside Ramupel and ", "zasitar": "Zasitar design beside Botuvik and ",
-             "ramupel": "Ramupel design beside ", "dopuvik": "Dopuvik design beside Zasitar and "}[args.design]
+             "ramupel": "Ramupel design beside ", "dopuvik": "Dopuvik design beside Zasitar and ",
+             "vomotar": "Vomotar design beside Dopuvik and "}[args.design]
     out = {"metric": f"prefill and decode tok/s of the {title}Llama at equal size (bf16)", "impl": "ours",
            "layers": layers, "batch": batch, "prompt_len": prompt, "prefill_len": prefill_len, "peaks": peaks, "sizes": {}}
     try:
@@ -283,6 +310,10 @@ def compare_designs(args, peaks) -> int:
                 designs = [("zasitar", zasitar_config(size, layers)), ("botuvik", botuvik_config(size, layers)), designs[1]]
             if dopuvik:
                 designs = [("dopuvik", dopuvik_config(size, layers)), ("zasitar", zasitar_config(size, layers)), designs[1]]
+            if vomotar:
+                designs = [("vomotar", vomotar_config(size, layers)), ("dopuvik", dopuvik_config(size, layers)), designs[1]]
+            if args.only:
+                designs = [d for d in designs if d[0] in args.only.split(",")]
             for name, raw in designs:
                 vocab = raw.get("vocab", raw.get("vocab_size"))
                 tmp = tempfile.mkdtemp(prefix="llmplayer_b200_bench_")
@@ -343,8 +374,10 @@ def compare_designs(args, peaks) -> int:
                 }
                 del engine, profiled
                 torch.cuda.empty_cache()
-            row["rooflines"] = {} if zasitar or dopuvik else hybrid_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len)
-            if dopuvik:
+            row["rooflines"] = {} if zasitar or dopuvik or vomotar else hybrid_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len)
+            if vomotar and "vomotar" in row:
+                row["rooflines"].update(vomotar_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
+            if "dopuvik" in row:
                 row["rooflines"].update(dopuvik_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
             if botuvik or zasitar:
                 row["rooflines"].update(botuvik_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
@@ -516,6 +549,38 @@ def dopuvik_rooflines(size, layers, row, peaks, batch, context, n):
     return out
 
 
+def vomotar_rooflines(size, layers, row, peaks, batch, context, n):
+    """The Vomotar kernels beside their Dopuvik (and Llama) twins (``dopuvik_rooflines``): prompt kernels against the bf16
+    tensor peak, decode and elementwise kernels against the copy bandwidth. Chunked attention's work counts the keys of a
+    query's own chunk only."""
+    width, heads, _, (gh, gk, gv), ff = HYBRID_SIZES[size]
+    n_pair = sum(1 for i in range(layers) if i % 4 == 0)
+    n_delta = layers - n_pair
+    flops, gbs = peaks["bf16_tflops"] * 1e12, peaks["hbm_gbs"] * 1e9
+    hd, G, W = width // heads, max(1, heads // 4), VOMOTAR_CHUNK
+    dense = (2 * ff // 3 + 127) // 128 * 128
+    pre, dec = row["vomotar"]["prefill_sections_ms"], row["vomotar"]["decode_sections_ms"]
+
+    def frac(work, ms, count, peak):
+        return None if not ms or not count else work / (ms / count / 1e3) / peak
+    seen = sum(i % W + 1 for i in range(n))                          # (query, key) pairs inside the chunks
+    return {
+        "prefill vomotar attention in chunks, keys seen (of tensor peak)": frac(
+            heads * seen * 4 * hd, pre.get("left.attention.scores"), n_pair, flops),
+        "prefill vomotar retention recurrence (of tensor peak)": frac(6.0 * gh * gk * gv * n, pre.get("right.recurrence.scan"), n_pair, flops),
+        "prefill vomotar delta-rule recurrence (of tensor peak)": frac(8.0 * gh * gk * gk * n, pre.get("recurrence.scan"), n_delta, flops),
+        "prefill vomotar short convolutions (of copy bandwidth)": frac(n * 3 * gh * gk * 8, pre.get("recurrence.conv"), n_delta, gbs),
+        "prefill vomotar low-rank gates (of copy bandwidth)": frac(n * 2 * gh * gk * 4, pre.get("recurrence.gates"), n_delta, gbs),
+        "prefill vomotar gate/up product (of tensor peak)": frac(2.0 * n * width * 2 * dense, pre.get("ffn.gate_up"), layers, flops),
+        "prefill vomotar two normed results summed (of copy bandwidth)": frac(n * width * (4 * 4 + 2), pre.get("mixer.sum"), n_pair, gbs),
+        "decode vomotar attention in chunks (of copy bandwidth)": frac(
+            batch * (context % W) * 2 * G * hd * 2, dec.get("left.attention.scores"), n_pair, gbs),
+        "decode vomotar retention recurrence (of copy bandwidth)": frac(batch * gh * gk * gv * 4 * 2, dec.get("right.recurrence.scan"), n_pair, gbs),
+        "decode vomotar delta-rule recurrence (of copy bandwidth)": frac(
+            batch * gh * gk * gk * 4 * 2, dec.get("recurrence.scan", dec.get("recurrence.step")), n_delta, gbs),
+    }
+
+
 def spread(values):
     return {"median": statistics.median(values), "min": min(values), "max": max(values), "repeats": len(values)}
 
@@ -536,10 +601,11 @@ def main() -> int:
     ap.add_argument("--prefill-only", action="store_true",
                     help="measure only the 2,048-token prefill (small runs for profiling)")
     ap.add_argument("--profile", action="store_true", help="add the device time per section of the model walk")
-    ap.add_argument("--design", default="llama", choices=("llama", "ramupel", "botuvik", "zasitar", "dopuvik"),
-                    help="ramupel / botuvik / zasitar / dopuvik: that design beside the closest others at equal size (another workload; see "
+    ap.add_argument("--design", default="llama", choices=("llama", "ramupel", "botuvik", "zasitar", "dopuvik", "vomotar"),
+                    help="ramupel / botuvik / zasitar / dopuvik / vomotar: that design beside the closest others at equal size (another workload; see "
                          "the module text)")
-    ap.add_argument("--size", default=None, choices=sorted(HYBRID_SIZES), help="with --design ramupel / botuvik / zasitar: one size only")
+    ap.add_argument("--size", default=None, choices=sorted(HYBRID_SIZES), help="with --design: one size only")
+    ap.add_argument("--only", default=None, help="with --design: only these of the designs beside each other (comma-separated)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -550,7 +616,7 @@ def main() -> int:
     if args.gpus != 1:
         print(f"bench.py measures one GPU; --gpus {args.gpus} is not supported by this single-GPU library")
         return 2
-    if args.design in ("ramupel", "botuvik", "zasitar", "dopuvik"):
+    if args.design in ("ramupel", "botuvik", "zasitar", "dopuvik", "vomotar"):
         return compare_designs(args, load_peaks())
     args.warmup = max(3, args.warmup)
     repeats = max(1, args.repeats)

@@ -85,7 +85,9 @@ __device__ __forceinline__ float rotated_channel(const float* head, int c, int r
 }
 constexpr int SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_OUTPUT = 2;
 
-template <int KP, int VT, int KPT, int JT>
+// EXTRA: rotation, fixed decays, and the delta rule with a decay per key channel (instantiations of their own, so that the
+// common forms carry none of it).
+template <int KP, int VT, int KPT, int JT, bool EXTRA>
 __global__ void __launch_bounds__(VT / JT * KP)
 gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ decay,
                 float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ q_start,
@@ -135,13 +137,17 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
         for (int e = tid; e < nt * dk; e += blockDim.x) {
             const int i = e / dk, c = e - i * dk;
             const float* row = proj + (long long)(tb + i) * ld;
-            const float* qh = row + q_off + (h / qk_group) * dk;
-            const float* kh = row + k_off + (h / qk_group) * dk;
-            const float2* cs = angles + (long long)(tb + i) * (rd >> 1);
-            qs[e] = (rd > 0 ? rotated_channel(qh, c, rd, interleaved, cs) : qh[c]) * q_scale;
-            ks[e] = (rd > 0 ? rotated_channel(kh, c, rd, interleaved, cs) : kh[c]) * (key_gain ? key_gain[(long long)(tb + i) * H + h] : 1.0f);
-            as[e] = decay_form == DECAY_FIXED ? decay[h]
-                    : decay_form == DECAY_HEAD ? decay[(long long)(tb + i) * H + h] : decay[((long long)(tb + i) * H + h) * dk + c];
+            const float gain = key_gain ? key_gain[(long long)(tb + i) * H + h] : 1.0f;
+            if (EXTRA && rd > 0) {
+                const float2* cs = angles + (long long)(tb + i) * (rd >> 1);
+                qs[e] = rotated_channel(row + q_off + (h / qk_group) * dk, c, rd, interleaved, cs) * q_scale;
+                ks[e] = rotated_channel(row + k_off + (h / qk_group) * dk, c, rd, interleaved, cs) * gain;
+            } else {
+                qs[e] = row[q_off + (h / qk_group) * dk + c] * q_scale;
+                ks[e] = row[k_off + (h / qk_group) * dk + c] * gain;
+            }
+            if (EXTRA && decay_form == DECAY_FIXED) as[e] = decay[h];
+            else as[e] = decay_form == DECAY_HEAD ? decay[(long long)(tb + i) * H + h] : decay[((long long)(tb + i) * H + h) * dk + c];
         }
         for (int e = tid; e < nt * VT; e += blockDim.x) {
             const int i = e / VT, c = e - i * VT;
@@ -165,7 +171,7 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, in
                 // Both read-outs are taken from the state before the token's write, S^T k and S^T q, in one pass of
                 // shuffles: o = S^T q + u (k . q) with the decayed S. One decay a per head comes out of the sums (the
                 // decayed S^T k is a (S^T k)); a decay per key channel is applied to the entries first.
-                const bool by_channel = decay_form == DECAY_CHANNEL;
+                const bool by_channel = EXTRA && decay_form == DECAY_CHANNEL;
                 float r1[JT], r2[JT], kq = 0.f;
 #pragma unroll
                 for (int jj = 0; jj < JT; ++jj) r1[jj] = r2[jj] = 0.f;
@@ -783,21 +789,27 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
     if (dk > 512) LP_REFUSE("gla_scan: %d key channels per head (supported: up to 512)", dk);
     if (q_off < 0 || k_off < 0 || v_off < 0 || q_off + qk_heads * dk > ld || k_off + qk_heads * dk > ld || v_off + H * (dv - (ones ? 1 : 0)) > ld)
         LP_REFUSE("gla_scan: slices at %d, %d, %d do not fit rows of %d", q_off, k_off, v_off, ld);
+    const bool extra = rd > 0 || decay_form == DECAY_FIXED || (beta && decay_form == DECAY_CHANNEL);
 #define LP_LAUNCH_SCAN(KP_, VT_, N, JT_)                                                                                 \
+    do {                                                                                                              \
+        if (extra) LP_LAUNCH_SCAN_FORM(KP_, VT_, N, JT_, true);                                                       \
+        else LP_LAUNCH_SCAN_FORM(KP_, VT_, N, JT_, false);                                                            \
+    } while (0)
+#define LP_LAUNCH_SCAN_FORM(KP_, VT_, N, JT_, EX_)                                                                                 \
     do {                                                                                                              \
         dim3 grid((dv + VT_ - 1) / VT_, H, B * chunks);                                                               \
         const size_t smem = ((size_t)3 * TB * dk + (size_t)TB * VT_) * sizeof(float);                                 \
         if (smem > 48 * 1024) {                                                                                       \
-            cudaError_t e = cudaFuncSetAttribute(gla_scan_kernel<KP_, VT_, N, JT_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(gla_scan_kernel<KP_, VT_, N, JT_, EX_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) LP_REFUSE("gla_scan: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e)); \
         }                                                                                                             \
         if (chunks == 1) {                                                                                            \
-            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
+            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_, EX_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_WHOLE, 1, 0, (float*)nullptr,       \
                       (float*)nullptr, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                               \
         } else {                                                                                                      \
             dim3 grid_local((state_cols + VT_ - 1) / VT_, H, B * chunks);                                             \
-            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid_local, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
+            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_, EX_>, grid_local, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_LOCAL, chunks, chunk, chunk_state,  \
                       chunk_decay, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                                   \
             const long long per = (long long)H * dv * dk;                                                             \
@@ -807,7 +819,7 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
             else                                                                                                      \
                 lp_launch(gla_combine_kernel, dim3((unsigned)((per + 255) / 256), B), 256, 0, stream, state, slots,   \
                           q_start, chunk_state, (const float*)chunk_decay, H, dk, dv, chunks, chunk);                 \
-            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
+            lp_launch(gla_scan_kernel<KP_, VT_, N, JT_, EX_>, grid, VT_ / JT_ * KP_, smem, stream, proj, ld, q_off, k_off, v_off,     \
                       decay, state, slots, q_start, out, H, dk, dv, q_scale, SCAN_OUTPUT, chunks, chunk, chunk_state, \
                       chunk_decay, decay_form, key_gain, ones, bonus, qk_group, beta, state_cols, (const float2*)angles, rd, interleaved);                                                                                   \
         }                                                                                                             \
@@ -822,6 +834,7 @@ extern "C" int lp_gla_scan(const float* proj, int ld, int q_off, int k_off, int 
     else if (dk <= 256) LP_LAUNCH_SCAN(16, 32, 16, 2);
     else LP_LAUNCH_SCAN(16, 16, 32, 1);
 #undef LP_LAUNCH_SCAN
+#undef LP_LAUNCH_SCAN_FORM
     return lp_check_launch("gla_scan");
 }
 

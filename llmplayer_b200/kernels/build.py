@@ -37,6 +37,7 @@ LIBRARIES: Dict[str, str] = {
     "latent_attention": "latent_attention.cu",
     "linear_attention": "linear_attention.cu",
     "routing": "routing.cu",
+    "chunked_recurrence": "chunked_recurrence.cu",
 }
 HEADERS = ("common.cuh", "attention_noalloc.h", "tcgen05_utils.cuh", "attention_decode.cuh")
 

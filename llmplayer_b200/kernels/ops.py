@@ -98,6 +98,13 @@ _SIGNATURES = {
         "lp_gla_finish": [_P, _P, _F, _P, _I, _P, _I, _I, _I, _I, _P, ctypes.c_longlong, _I, _I, _I, _P, _P],
         "lp_exp_gates": [_P, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _P],
     },
+    "chunked_recurrence": {
+        "lp_chunked_tokens": [],
+        "lp_chunked_record_floats": [_I, _I],
+        "lp_chunked_value_floats": [_I],
+        "lp_chunked_recurrence": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
+                                  _P, _P, _P],
+    },
     "host_loop": {
         "lp_decode_loop": [_P, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P],
         "lp_decode_loop_sampled": [_P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P,
@@ -1353,6 +1360,9 @@ def gla_decay(low: torch.Tensor, up: torch.Tensor, bias: Optional[torch.Tensor],
 
 GLA_CHUNK = 128               # tokens per chunk of a long prompt's recurrence
 GLA_CHUNKED_FROM = 256        # from how many new tokens of a sequence on the chunks run side by side
+CHUNKED_FROM = 32             # from how many new tokens on the chunks' sums run as tensor-core products (where asked for)
+CHUNKED_MAX_KEYS = 256
+CHUNKED_BUFFER_BYTES = 256 << 20   # room for the chunks' records; steps that need more run in several rounds
 
 
 def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, state: torch.Tensor,
@@ -1360,7 +1370,7 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
              value_dim: int, q_scale: float, max_new: int = 0, scratch=None, decay_per_head: bool = False,
              key_gain: Optional[torch.Tensor] = None, ones_column: bool = False,
              bonus: Optional[torch.Tensor] = None, qk_heads: Optional[int] = None,
-             delta_strength: Optional[torch.Tensor] = None, decay_fixed: bool = False, rotation: Optional["Rotation"] = None,
+             delta_strength: Optional[torch.Tensor] = None, tensor_cores: bool = False, decay_fixed: bool = False, rotation: Optional["Rotation"] = None,
              angles: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The recurrence S <- diag(decay_t) S + k_t v_t^T, out_t = S^T (q_t * q_scale) over the step's tokens of every
     sequence, from and into ``state`` float32 [slots, H, dv, dk] (row ``slots[b]`` for sequence b; a value column's
@@ -1382,7 +1392,9 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     chunks side by side here too (a chunk's effect on the state that enters it is S -> P S + L with a [dk, dk] matrix P,
     which the first pass forms beside L). ``decay_fixed``: ``decay`` is float32 [H], one constant per head. ``rotation``
     with ``angles`` (float32 [T, rotary_dim / 2, 2], cosines and sines of the step's tokens): queries and keys are rotated
-    as they are read."""
+    as they are read. ``tensor_cores``: steps with ``CHUNKED_FROM`` new tokens or more of a sequence run in chunks of 32
+    tokens whose sums are tensor-core products at float32 precision (csrc/chunked_recurrence.cu), for the forms without
+    ``bonus`` and ``ones_column``."""
     _want(proj, "gla_scan proj", torch.float32, 2)
     _want(decay, "gla_scan decay", torch.float32, 1 if decay_fixed else 2)
     _want(state, "gla_scan state", torch.float32, 4)
@@ -1418,6 +1430,23 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
             raise KernelError(f"gla_scan: angles {tuple(angles.shape)} for {T} tokens and {rd} channels")
     if qk_heads is not None and (qk_heads <= 0 or H % qk_heads):
         raise KernelError(f"gla_scan: {H} heads over {qk_heads} query / key heads")
+    form = 2 if decay_fixed else 1 if decay_per_head else 0
+    if (tensor_cores and scratch is not None and max_new >= CHUNKED_FROM and bonus is None and not ones_column
+            and dk <= CHUNKED_MAX_KEYS):
+        lib = library("chunked_recurrence")
+        delta = 1 if delta_strength is not None else 0
+        rec, val = lib.lp_chunked_record_floats(dk, delta), lib.lp_chunked_value_floats(dv)
+        total = -(-max_new // lib.lp_chunked_tokens())
+        room = min(total, max(1, CHUNKED_BUFFER_BYTES // (4 * B * H * (rec + val))))
+        records = scratch("chunk_records", (B * room * H * rec,), torch.float32)
+        values = scratch("chunk_values", (B * room * H * val,), torch.float32)
+        _check(lib, lib.lp_chunked_recurrence(
+            proj.data_ptr(), proj.shape[1], int(q_off), int(k_off), int(v_off), decay.data_ptr(), form, _ptr(key_gain),
+            _ptr(delta_strength), _ptr(angles) if rd else None, rd, interleaved, float(q_scale), state.data_ptr(),
+            slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), B, H, dk, dv, int(qk_heads or H), int(max_new), room,
+            records.data_ptr(), values.data_ptr(), _stream()))
+        count_launches(2 * -(-total // room) - 1)
+        return out
     chunks, chunk_state, chunk_decay = 1, None, None
     # the delta rule's passes are bound by their chain of tokens, not by arithmetic: shorter chunks, more of them
     # (measured at 4 heads of 64 x 64 over 2,048 tokens: chunks of 128 / 64 / 32: 0.28 / 0.22 / 0.34 ms; the chunks'
@@ -1432,7 +1461,7 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torc
     _check(lib, lib.lp_gla_scan(proj.data_ptr(), proj.shape[1], int(q_off), int(k_off), int(v_off), decay.data_ptr(),
                                 state.data_ptr(), slots.data_ptr(), q_start.data_ptr(), out.data_ptr(), B, H, dk, dv,
                                 float(q_scale), chunks, chunk, _ptr(chunk_state), _ptr(chunk_decay),
-                                2 if decay_fixed else 1 if decay_per_head else 0, _ptr(key_gain), 1 if ones_column else 0,
+                                form, _ptr(key_gain), 1 if ones_column else 0,
                                 _ptr(bonus), int(qk_heads or H), _ptr(delta_strength), _ptr(angles) if rd else None, rd,
                                 interleaved, _stream()))
     if chunks > 1:

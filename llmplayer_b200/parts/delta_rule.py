@@ -69,12 +69,12 @@ class GatedDeltaRule(Part):
             s.strength: TensorSpec((H, d), MATRIX),
             s.a_log: TensorSpec((H,), BIAS),
             s.out_norm: TensorSpec((s.value_dim,), GAIN),
-            s.decay: TensorSpec((H if s.decay_up is None else ANY, d), MATRIX),
+            s.decay: TensorSpec((H if s.decay_up is None else ANY, d), MATRIX, fill=s.key_dim),
             s.dt_bias: TensorSpec((H if s.decay_up is None else H * s.key_dim,), BIAS),
-            s.gate: TensorSpec((self.values if s.gate_up is None else ANY, d), MATRIX),
+            s.gate: TensorSpec((self.values if s.gate_up is None else ANY, d), MATRIX, fill=s.key_dim),
             s.o: TensorSpec((d, self.values), MATRIX),
-            **({s.decay_up: TensorSpec((H * s.key_dim, ANY), MATRIX)} if s.decay_up is not None else {}),
-            **({s.gate_up: TensorSpec((self.values, ANY), MATRIX)} if s.gate_up is not None else {}),
+            **({s.decay_up: TensorSpec((H * s.key_dim, ANY), MATRIX, fill=s.key_dim)} if s.decay_up is not None else {}),
+            **({s.gate_up: TensorSpec((self.values, ANY), MATRIX, fill=s.key_dim)} if s.gate_up is not None else {}),
         }
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
@@ -161,7 +161,7 @@ class GatedDeltaRule(Part):
         with ops.section("recurrence.scan"):
             ops.gla_scan(mixed, 0, self.qk, 2 * self.qk, decay, state, ctx.slots, ctx.q_start, raw, num_heads=H,
                          key_dim=dk, value_dim=dv, q_scale=1.0, max_new=ctx.max_new, scratch=ctx.buffer,
-                         decay_per_head=not by_channel, qk_heads=G, delta_strength=strength)
+                         decay_per_head=not by_channel, qk_heads=G, delta_strength=strength, tensor_cores=rt.fast)
         o = ctx.buffer("attn_out", (T, self.values), rt.act_dtype)
         with ops.section("recurrence.norm"):
             clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None

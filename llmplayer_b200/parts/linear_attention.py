@@ -96,7 +96,7 @@ class GatedLinearAttention(Part):
         raw = ctx.buffer("gla_raw", (T, H * dv), torch.float32)
         with ops.section("recurrence.scan"):
             ops.gla_scan(proj, q_off, k_off, v_off, decay, cache.rows, ctx.slots, ctx.q_start, raw, num_heads=H,
-                         key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, max_new=ctx.max_new, scratch=ctx.buffer)
+                         key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, max_new=ctx.max_new, scratch=ctx.buffer, tensor_cores=rt.fast)
         o = ctx.buffer("attn_out", (T, H * dv), rt.act_dtype)
         # an output product that sums partial results into `out` wants it zero: the kernel before it clears it
         clear = self.out.sums_into(ctx, T, "mixer_out", ops.STORE)

@@ -109,7 +109,7 @@ class Retention(Part):
             ops.gla_scan(proj, offset, offset + self.keys, v_off, self.decays, cache.rows, ctx.slots, ctx.q_start, raw,
                          num_heads=H, key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, max_new=ctx.max_new,
                          scratch=ctx.buffer, decay_fixed=True, rotation=rotation,
-                         angles=ctx.angles(rotation) if rotation.rotary_dim else None)
+                         angles=ctx.angles(rotation) if rotation.rotary_dim else None, tensor_cores=rt.fast)
         o = ctx.buffer("attn_out", (T, self.values), rt.act_dtype)
         with ops.section("recurrence.norm"):
             # an output product that sums partial results wants its target zero: this kernel clears it on the side

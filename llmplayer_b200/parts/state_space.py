@@ -110,7 +110,7 @@ class StateSpace(Part):
         with ops.section("recurrence.scan"):
             ops.gla_scan(mixed, inner + G * N, inner, 0, gates[0], state, ctx.slots, ctx.q_start, raw, num_heads=H,
                          key_dim=N, value_dim=P, q_scale=1.0, max_new=ctx.max_new, scratch=ctx.buffer,
-                         decay_per_head=True, key_gain=gates[1], qk_heads=G)
+                         decay_per_head=True, key_gain=gates[1], qk_heads=G, tensor_cores=rt.fast)
         o = ctx.buffer("attn_out", (T, inner), rt.act_dtype)
         with ops.section("recurrence.norm"):
             # an output product that sums partial results wants its target zero: this kernel clears it on the side
