@@ -584,6 +584,97 @@ short_conv_kernel(const float* __restrict__ in, int ldi, const TW* __restrict__ 
     }
 }
 
+// The same with silu, where the first `heads` * dim channels are heads that become unit vectors behind it (x / sqrt(sum x^2 +
+// eps), the first `scaled` heads also times `scale`). A block takes whole heads (`per_block` of them, `head_warps` warps each)
+// or, behind them, as many single channels as it has threads; a thread keeps its channel's 32 outputs in registers, and a
+// warp's sums over its channels meet in a transposing reduction that leaves token t's sum in lane t.
+__global__ void __launch_bounds__(512)
+conv_unit_heads_kernel(const float* __restrict__ in, int ldi, const float* __restrict__ taps, float* __restrict__ tail,
+                       const int* __restrict__ slots, const int* __restrict__ q_start, float* __restrict__ out, int ldo, int C, int K,
+                       int heads, int dim, int head_warps, int per_block, int head_blocks, float eps, float scale, int scaled) {
+    __shared__ float part[16][CONV_CHUNK], factor[16][CONV_CHUNK];
+    lp_grid_release();
+    lp_grid_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool unit = (int)blockIdx.x < head_blocks;
+    const int slot_in = warp / head_warps;                     // which of the block's heads
+    const int head = blockIdx.x * per_block + slot_in, within = (warp - slot_in * head_warps) * 32 + lane;
+    const int c = unit ? head * dim + within : heads * dim + (blockIdx.x - head_blocks) * blockDim.x + threadIdx.x;
+    const bool valid = unit ? head < heads && within < dim : c < C;
+    const int b = blockIdx.z;
+    const int t0 = q_start[b], t1 = q_start[b + 1];
+    const int begin = t0 + blockIdx.y * CONV_CHUNK;
+    if (begin >= t1) return;                                    // the whole block
+    const int n = min(t1 - begin, CONV_CHUNK);
+    float y[CONV_CHUNK];
+#pragma unroll
+    for (int i = 0; i < CONV_CHUNK; ++i) y[i] = 0.f;
+    if (valid) {
+        float w[CONV_MAX_TAPS], hist[CONV_MAX_TAPS - 1];
+#pragma unroll
+        for (int j = 0; j < CONV_MAX_TAPS; ++j) {
+            const int tap = j - (CONV_MAX_TAPS - K);
+            w[j] = tap >= 0 ? taps[(long long)c * K + tap] : 0.f;
+        }
+        float* keep = tail + (long long)slots[b] * (K - 1) * C + c;
+#pragma unroll
+        for (int i = 0; i < CONV_MAX_TAPS - 1; ++i) {
+            float v = 0.f;
+            if (i < K - 1) {
+                const int src = begin - 1 - i;
+                v = src >= t0 ? in[(long long)src * ldi + c] : keep[(long long)(K - 1 + src - t0) * C];
+            }
+            hist[CONV_MAX_TAPS - 2 - i] = v;
+        }
+        if (begin == t0) {                                      // the step's last K - 1 inputs become the tail, as above
+            for (int j = 0; j < K - 1; ++j) {
+                const int src = t1 - (K - 1) + j;
+                keep[(long long)j * C] = src >= t0 ? in[(long long)src * ldi + c] : keep[(long long)(j + t1 - t0) * C];
+            }
+        }
+        float x[CONV_CHUNK];
+#pragma unroll
+        for (int i = 0; i < CONV_CHUNK; ++i) x[i] = i < n ? __ldg(in + (long long)(begin + i) * ldi + c) : 0.f;
+#pragma unroll
+        for (int i = 0; i < CONV_CHUNK; ++i) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) {
+                const int at = i - (CONV_MAX_TAPS - 1) + j;     // the input 7 - j tokens back
+                acc = fmaf(w[j], at >= 0 ? x[at >= 0 ? at : 0] : hist[at + CONV_MAX_TAPS - 1 < CONV_MAX_TAPS - 1 ? at + CONV_MAX_TAPS - 1 : 0], acc);
+            }
+            acc = fmaf(w[CONV_MAX_TAPS - 1], x[i], acc);
+            y[i] = i < n ? acc / (1.0f + expf(-acc)) : 0.f;
+        }
+    }
+    if (unit) {
+        float v[CONV_CHUNK];
+#pragma unroll
+        for (int i = 0; i < CONV_CHUNK; ++i) v[i] = y[i] * y[i];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const bool up = lane & o;
+#pragma unroll
+            for (int i = 0; i < o; ++i) {
+                const float give = up ? v[i] : v[i + o], own = up ? v[i + o] : v[i];
+                v[i] = own + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+        }
+        part[warp][lane] = v[0];
+        __syncthreads();
+        if (within < 32) {                                      // the first warp of every head
+            float ss = 0.f;
+            for (int k = 0; k < head_warps; ++k) ss += part[slot_in * head_warps + k][lane];
+            factor[slot_in][lane] = (head < scaled ? scale : 1.0f) / sqrtf(ss + eps);
+        }
+        __syncthreads();
+    }
+    if (!valid) return;
+#pragma unroll
+    for (int i = 0; i < CONV_CHUNK; ++i)
+        if (i < n) out[(long long)(begin + i) * ldo + c] = unit ? y[i] * factor[slot_in][i] : y[i];
+}
+
 __device__ __forceinline__ float lp_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---------------------------------------------------------------- step sizes, decays and write strengths of a recurrence
@@ -613,7 +704,7 @@ decay_gates_kernel(const float* __restrict__ proj, int ld, int z_off, int b_off,
 //   decays: decay[c] = exp(-exp(a_log[c / dk]) * softplus(z[c] + dt_bias[c]))  (no clamp; one a_log per head of dk channels)
 //   gate:   out[c] = z[c]                                                      (the reader applies its activation)
 //   strength[h] = sigmoid(zb[h])
-// A CTA takes 64 tokens x 64 channels of one of the two maps, 4 x 4 sums per thread; the CTAs of the first column also
+// A CTA takes 128 tokens x 64 channels of one of the two maps, 8 x 4 sums per thread; the CTAs of the first column also
 // write their tokens' strengths. grid (column tiles of both maps, token tiles).
 struct RankMap {
     int off, rank, channels;      // columns [off, off + rank) of the projection -> `channels` outputs
@@ -621,64 +712,84 @@ struct RankMap {
     int up_bf16;
     float* out;                   // [T, channels]
 };
-constexpr int RM_TILE = 64, RM_K = 32;
+constexpr int RM_TOKENS = 128, RM_TILE = 64, RM_K = 32;
 
 __global__ void __launch_bounds__(256)
 low_rank_gates_kernel(const float* __restrict__ proj, int ld, int T, int H, RankMap a, const float* __restrict__ dt_bias,
                       const float* __restrict__ a_log, int dk, RankMap g, int a_tiles, int b_off, float* __restrict__ strength) {
-    __shared__ float low[RM_TILE][RM_K + 1], up[RM_TILE][RM_K + 1];
+    __shared__ float low[RM_K][RM_TOKENS + 4], up[RM_K][RM_TILE + 4];
     lp_grid_release();
     lp_grid_wait();
-    const int t0 = blockIdx.y * RM_TILE;
+    const int t0 = blockIdx.y * RM_TOKENS;
     const bool decays = (int)blockIdx.x < a_tiles;
     const RankMap m = decays ? a : g;
     const int c0 = (decays ? blockIdx.x : blockIdx.x - a_tiles) * RM_TILE;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float acc[4][4];
+    float acc[8][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    const int lr = threadIdx.x % RM_K, li = threadIdx.x / RM_K;          // a thread loads column lr of every eighth row
     for (int r0 = 0; r0 < m.rank; r0 += RM_K) {
-        for (int e = threadIdx.x; e < RM_TILE * RM_K; e += 256) {
-            const int i = e / RM_K, r = r0 + e % RM_K;
-            const bool in = r < m.rank;
-            low[i][e % RM_K] = (in && t0 + i < T) ? proj[(long long)(t0 + i) * ld + m.off + r] : 0.f;
-            float w = 0.f;
-            if (in && c0 + i < m.channels) {
-                const long long at = (long long)(c0 + i) * m.rank + r;
-                w = m.up_bf16 ? __bfloat162float(((const __nv_bfloat16*)m.up)[at]) : ((const float*)m.up)[at];
-            }
-            up[i][e % RM_K] = w;
+        const bool in = r0 + lr < m.rank;
+        float x[RM_TOKENS / 8], w[RM_TILE / 8];
+#pragma unroll
+        for (int u = 0; u < RM_TOKENS / 8; ++u) {
+            const int t = t0 + li + 8 * u;
+            x[u] = (in && t < T) ? __ldg(proj + (long long)t * ld + m.off + r0 + lr) : 0.f;
         }
+#pragma unroll
+        for (int u = 0; u < RM_TILE / 8; ++u) {
+            const int c = c0 + li + 8 * u;
+            const long long at = (long long)c * m.rank + r0 + lr;
+            w[u] = 0.f;
+            if (in && c < m.channels) w[u] = m.up_bf16 ? __bfloat162float(((const __nv_bfloat16*)m.up)[at]) : ((const float*)m.up)[at];
+        }
+        __syncthreads();
+#pragma unroll
+        for (int u = 0; u < RM_TOKENS / 8; ++u) low[lr][li + 8 * u] = x[u];
+#pragma unroll
+        for (int u = 0; u < RM_TILE / 8; ++u) up[lr][li + 8 * u] = w[u];
         __syncthreads();
 #pragma unroll 8
         for (int r = 0; r < RM_K; ++r) {
-            float x[4], w[4];
+            const float4 xa = *reinterpret_cast<const float4*>(&low[r][ty * 8]), xb = *reinterpret_cast<const float4*>(&low[r][ty * 8 + 4]);
+            const float4 wv = *reinterpret_cast<const float4*>(&up[r][tx * 4]);
+            const float xs[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { x[i] = low[ty + 16 * i][r]; w[i] = up[tx + 16 * i][r]; }
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+            for (int i = 0; i < 8; ++i) {
+                acc[i][0] = fmaf(xs[i], wv.x, acc[i][0]);
+                acc[i][1] = fmaf(xs[i], wv.y, acc[i][1]);
+                acc[i][2] = fmaf(xs[i], wv.z, acc[i][2]);
+                acc[i][3] = fmaf(xs[i], wv.w, acc[i][3]);
+            }
         }
-        __syncthreads();
     }
+    float rate[4], bias[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int t = t0 + ty + 16 * i;
-        if (t >= T) continue;
+    for (int j = 0; j < 4; ++j) {
+        const int c = c0 + tx * 4 + j;
+        rate[j] = decays && c < m.channels ? expf(a_log[c / dk]) : 0.f;
+        bias[j] = decays && c < m.channels ? dt_bias[c] : 0.f;
+    }
+    const bool quads = (m.channels & 3) == 0;                            // the outputs' rows are then aligned to 16 bytes
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int c = c0 + tx + 16 * j;
-            if (c >= m.channels) continue;
-            float v = acc[i][j];
-            if (decays) v = expf(-expf(a_log[c / dk]) * lp_softplus(v + dt_bias[c]));
-            m.out[(long long)t * m.channels + c] = v;
-        }
+    for (int i = 0; i < 8; ++i) {
+        const int t = t0 + ty * 8 + i, c = c0 + tx * 4;
+        if (t >= T || c >= m.channels) continue;
+        if (decays)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] = expf(-rate[j] * lp_softplus(acc[i][j] + bias[j]));
+        float* at = m.out + (long long)t * m.channels + c;
+        if (quads) *reinterpret_cast<float4*>(at) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        else
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (c + j < m.channels) at[j] = acc[i][j];
     }
     if (blockIdx.x == 0) {
-        for (int e = threadIdx.x; e < RM_TILE * H; e += 256) {
+        for (int e = threadIdx.x; e < RM_TOKENS * H; e += 256) {
             const int t = t0 + e / H, h = e % H;
             if (t < T) strength[(long long)t * H + h] = 1.0f / (1.0f + expf(-proj[(long long)t * ld + b_off + h]));
         }
@@ -905,6 +1016,24 @@ extern "C" int lp_short_conv(const float* in, int ldi, const void* taps, int w_d
     return lp_check_launch("short_conv");
 }
 
+// in: float32 [T, ldi] (C channels from the given pointer), the first heads * dim of them heads that become unit vectors behind
+// the convolution and silu; taps: float32 [C, K]; tail: float32 [slots, K - 1, C]; out: float32 [T, ldo].
+extern "C" int lp_conv_unit_heads(const float* in, int ldi, const float* taps, float* tail, const int* slots, const int* q_start,
+                                  float* out, int ldo, int B, int max_new, int C, int K, int heads, int dim, float eps, float scale,
+                                  int scaled, cudaStream_t stream) {
+    if (B <= 0 || max_new <= 0 || C <= 0) return 0;
+    if (K < 1 || K > CONV_MAX_TAPS) LP_REFUSE("conv_unit_heads: %d taps (supported: 1..%d)", K, CONV_MAX_TAPS);
+    if (ldi < C || ldo < C || heads <= 0 || dim <= 0 || dim > 512 || heads * dim > C) LP_REFUSE("conv_unit_heads: %d heads of %d in %d channels", heads, dim, C);
+    const int chunks = (max_new + CONV_CHUNK - 1) / CONV_CHUNK;
+    if (chunks > 65535 || B > 65535) LP_REFUSE("conv_unit_heads: %d chunks of tokens, %d sequences exceed the grid", chunks, B);
+    const int head_warps = (dim + 31) / 32, per_block = head_warps >= 4 ? 1 : 4 / head_warps;
+    const int threads = head_warps * per_block * 32;
+    const int head_blocks = (heads + per_block - 1) / per_block, rest = (C - heads * dim + threads - 1) / threads;
+    lp_launch(conv_unit_heads_kernel, dim3(head_blocks + rest, chunks, B), threads, 0, stream, in, ldi, taps, tail, slots, q_start, out, ldo,
+              C, K, heads, dim, head_warps, per_block, head_blocks, eps, scale, scaled);
+    return lp_check_launch("conv_unit_heads");
+}
+
 // proj: float32 [T, ld]; z_off: column of the H step-size pre-activations; b_off: column of the H write-strength
 // pre-activations (used only with `strength`); decay, dt_out (optional), strength (optional): float32 [T, H].
 extern "C" int lp_decay_gates(const float* proj, int ld, int z_off, int b_off, const float* dt_bias, const float* a_log,
@@ -932,7 +1061,8 @@ extern "C" int lp_low_rank_gates(const float* proj, int ld, int T, int H, int dk
     const RankMap a{a_off, a_rank, H * dk, a_up, a_dtype == LP_BF16, decay};
     const RankMap g{g_off, g_rank, g_up ? g_channels : 0, g_up, g_dtype == LP_BF16, gate};
     const int a_tiles = (a.channels + RM_TILE - 1) / RM_TILE, g_tiles = (g.channels + RM_TILE - 1) / RM_TILE;
-    const int rows = (T + RM_TILE - 1) / RM_TILE;
+    if ((((uintptr_t)decay | (uintptr_t)gate) & 15) != 0) LP_REFUSE("low_rank_gates: outputs must be aligned to 16 bytes");
+    const int rows = (T + RM_TOKENS - 1) / RM_TOKENS;
     if (rows > 65535) LP_REFUSE("low_rank_gates: %d tokens exceed the grid", T);
     lp_launch(low_rank_gates_kernel, dim3(a_tiles + g_tiles, rows), 256, 0, stream, proj, ld, T, H, a, dt_bias, a_log, dk, g, a_tiles,
               b_off, strength);

@@ -91,6 +91,7 @@ _SIGNATURES = {
         "lp_gla_scan": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P],
         "lp_low_rank_gates": [_P, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _P, _I, _P, _P],
         "lp_short_conv": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+        "lp_conv_unit_heads": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
         "lp_decay_gates": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _P],
         "lp_head_unit_norm": [_P, _I, _I, _I, _I, _F, _F, _I, _I, _P],
         "lp_gated_part_norm": [_P, _P, _I, _P, _P, _I, _P, _F, _P, _I, _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
@@ -104,6 +105,10 @@ _SIGNATURES = {
         "lp_chunked_value_floats": [_I],
         "lp_chunked_recurrence": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
                                   _P, _P, _P],
+    },
+    "delta_step": {
+        "lp_delta_step": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _F, _F, _P, _P, _P, _I, _P, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I,
+                          _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
     },
     "host_loop": {
         "lp_decode_loop": [_P, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P],
@@ -1530,6 +1535,28 @@ def short_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor]
     return out
 
 
+def conv_unit_heads(x: torch.Tensor, taps: torch.Tensor, tail: torch.Tensor, slots: torch.Tensor, q_start: torch.Tensor,
+                    out: torch.Tensor, *, max_new: int, heads: int, dim: int, eps: float, scale: float, scaled_heads: int) -> torch.Tensor:
+    """:func:`short_conv` with silu over all channels of ``x`` and :func:`head_unit_norm` over the first ``heads`` heads of
+    ``dim`` channels (the first ``scaled_heads`` also times ``scale``), in one kernel. ``taps``: float32."""
+    xp, ldx = _slice(x, "conv_unit_heads x")
+    op, ldo = _slice(out, "conv_unit_heads out")
+    _want(taps, "conv_unit_heads taps", torch.float32, 2)
+    _want(tail, "conv_unit_heads tail", torch.float32, 3)
+    _want(slots, "conv_unit_heads slots", torch.int32, 1)
+    _want(q_start, "conv_unit_heads q_start", torch.int32, 1)
+    T, C = x.shape
+    K = taps.shape[1]
+    B = slots.numel()
+    if taps.shape[0] != C or out.shape != x.shape or tail.shape[1:] != (K - 1, C) or q_start.numel() != B + 1:
+        raise KernelError(f"conv_unit_heads: x {tuple(x.shape)}, taps {tuple(taps.shape)}, tail {tuple(tail.shape)}, out "
+                          f"{tuple(out.shape)}, {B} sequences")
+    lib = library("linear_attention")
+    _check(lib, lib.lp_conv_unit_heads(xp, ldx, taps.data_ptr(), tail.data_ptr(), slots.data_ptr(), q_start.data_ptr(), op, ldo, B,
+                                       int(max_new), C, K, int(heads), int(dim), float(eps), float(scale), int(scaled_heads), _stream()))
+    return out
+
+
 def decay_gates(proj: torch.Tensor, z_off: int, dt_bias: Optional[torch.Tensor], a_log: torch.Tensor, decay: torch.Tensor,
                 dt: Optional[torch.Tensor] = None, strength: Optional[torch.Tensor] = None, b_off: int = 0) -> None:
     """Per token and head, from float32 columns of ``proj``: step = softplus(proj[:, z_off + h] + dt_bias[h]) (no
@@ -1585,6 +1612,50 @@ def low_rank_gates(proj: torch.Tensor, a_off: int, a_up: torch.Tensor, dt_bias: 
         proj.data_ptr(), proj.shape[1], T, H, int(key_dim), int(a_off), a_up.shape[1], a_up.data_ptr(), _code(a_up, "low_rank_gates a_up"),
         dt_bias.data_ptr(), a_log.data_ptr(), decay.data_ptr(), int(g_off), rank_g, channels, _ptr(g_up), code, _ptr(gate),
         int(b_off), strength.data_ptr(), _stream()))
+
+
+def delta_step(proj: torch.Tensor, columns, taps: torch.Tensor, tail: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+               dt_bias: torch.Tensor, a_log: torch.Tensor, gain: torch.Tensor, norm_eps: float, out: torch.Tensor, *,
+               num_heads: int, qk_heads: int, key_dim: int, value_dim: int, unit_eps: float, q_scale: float,
+               a_up: Optional[torch.Tensor] = None, g_up: Optional[torch.Tensor] = None, gate_sigmoid: bool = False,
+               clear: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One token for each sequence through a delta-rule layer, from the projection of its input to the input of its output
+    product, in one kernel (csrc/delta_step.cu): what :func:`short_conv`, :func:`head_unit_norm`, :func:`decay_gates` or
+    :func:`low_rank_gates`, :func:`gla_scan` and :func:`gla_finish` do for a step of several tokens. ``proj``: float32 [B, F];
+    ``columns`` = (first convolution channel [q | k | v], write strengths, decays, gate); ``out``: [B, H * dv]. ``a_up``
+    [H * dk, rank] / ``g_up`` [H * dv, rank]: the decays' / the gate's low-rank maps (``dt_bias`` is then [H * dk])."""
+    _want(proj, "delta_step proj", torch.float32, 2)
+    _want(taps, "delta_step taps", torch.float32, 2)
+    _want(tail, "delta_step tail", torch.float32, 3)
+    _want(state, "delta_step state", torch.float32, 4)
+    _want(slots, "delta_step slots", torch.int32, 1)
+    _want(dt_bias, "delta_step dt_bias", torch.float32, 1)
+    _want(a_log, "delta_step a_log", torch.float32, 1)
+    _want(gain, "delta_step gain", torch.float32, 1)
+    _want(out, "delta_step out", ndim=2)
+    B, H, G, dk, dv = slots.numel(), num_heads, qk_heads, key_dim, value_dim
+    channels, K = taps.shape
+    if (proj.shape[0] != B or channels != 2 * G * dk + H * dv or tail.shape[1:] != (K - 1, channels) or state.shape[1:] != (H, dv, dk)
+            or out.shape != (B, H * dv) or a_log.numel() != H or gain.numel() != dv or dt_bias.numel() != (H if a_up is None else H * dk)):
+        raise KernelError(f"delta_step: proj {tuple(proj.shape)}, taps {tuple(taps.shape)}, tail {tuple(tail.shape)}, state "
+                          f"{tuple(state.shape)}, out {tuple(out.shape)}, {B} sequences, {H} heads on {G} of {dk} x {dv}")
+    code, ranks = F32, [0, 0]
+    for i, (name, up, rows) in enumerate((("a_up", a_up, H * dk), ("g_up", g_up, H * dv))):
+        if up is not None:
+            _want(up, f"delta_step {name}", ndim=2)
+            code, ranks[i] = _code(up, f"delta_step {name}"), up.shape[1]
+            if up.shape[0] != rows:
+                raise KernelError(f"delta_step: {name} {tuple(up.shape)} for {rows} rows")
+    if a_up is not None and g_up is not None and a_up.dtype != g_up.dtype:
+        raise KernelError("delta_step: both low-rank maps have one number format")
+    c_off, b_off, a_off, g_off = (int(c) for c in columns)
+    lib = library("delta_step")
+    _check(lib, lib.lp_delta_step(
+        proj.data_ptr(), proj.shape[1], c_off, b_off, a_off, g_off, taps.data_ptr(), tail.data_ptr(), K, float(unit_eps), float(q_scale),
+        dt_bias.data_ptr(), a_log.data_ptr(), _ptr(a_up), ranks[0], _ptr(g_up), ranks[1], code, 1 if gate_sigmoid else 0, gain.data_ptr(),
+        float(norm_eps), state.data_ptr(), slots.data_ptr(), out.data_ptr(), _code(out, "delta_step out"), B, H, G, dk, dv,
+        *_clear_args(clear, "delta_step"), _stream()))
+    return out
 
 
 def head_unit_norm(x: torch.Tensor, offset: int, heads: int, dim: int, eps: float, scale: float = 1.0,

@@ -93,6 +93,10 @@ class GatedDeltaRule(Part):
                 raise WeightError(f"{down} has {tensors[down].shape[0]} rows but {up} has {tensors[up].shape[1]} columns")
         self.decay_up = runtime.matrix(tensors[s.decay_up]) if s.decay_up is not None else None
         self.gate_up = runtime.matrix(tensors[s.gate_up]) if s.gate_up is not None else None
+        if self.decay_up is not None and self.gate_up is not None and self.decay_up.dtype != self.gate_up.dtype:
+            self.decay_up, self.gate_up = self.decay_up.float(), self.gate_up.float()       # mixed storage: widen
+        # one token per sequence in one kernel, a CTA per query / key head; with many value heads on one it would be slow
+        self.step_kernel = s.num_heads // s.num_qk_heads <= 4 and s.value_dim * 3 + s.key_dim * 3 + self.decay_rows + self.gate_rows <= 11000
         self.taps = runtime.gain(torch.cat([tensors[n].to(torch.float32) for n in (s.q_conv, s.k_conv, s.v_conv)], dim=0))
         self.a_log = runtime.gain(tensors[s.a_log])
         self.dt_bias = runtime.gain(tensors[s.dt_bias])
@@ -140,10 +144,37 @@ class GatedDeltaRule(Part):
         a_off = b_off + H
         g_off = a_off + self.decay_rows
         state, tail = cache.blocks
+        o = ctx.buffer("attn_out", (T, self.values), rt.act_dtype)
+        clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None
+        if ctx.all_single and self.step_kernel:
+            with ops.section("recurrence.step"):
+                ops.delta_step(proj, (offset, b_off, a_off, g_off), self.taps, tail, state, ctx.slots, self.dt_bias, self.a_log,
+                               self.out_gain, s.norm_eps, o, num_heads=H, qk_heads=G, key_dim=dk, value_dim=dv, unit_eps=UNIT_EPS,
+                               q_scale=float(dk) ** -0.5, a_up=self.decay_up, g_up=self.gate_up,
+                               gate_sigmoid=s.gate_activation == "sigmoid", clear=clear)
+        else:
+            self._recur(ctx, proj, offset, state, tail, o, clear)
+        if clear is not None:
+            ctx.note_cleared()
+        with ops.section("recurrence.out"):
+            if overwrite:
+                self.out.store(o, residual, ctx)
+                return False
+            return self.out.accumulate(o, residual, ctx, then_norm)
+
+    def _recur(self, ctx, proj: torch.Tensor, offset: int, state: torch.Tensor, tail: torch.Tensor, o: torch.Tensor, clear) -> None:
+        """From the input projections to the normed and gated heads ``o``, for steps with several tokens of a sequence."""
+        s, rt = self.spec, self.runtime
+        T = proj.shape[0]
+        H, G, dk, dv = s.num_heads, s.num_qk_heads, s.key_dim, s.value_dim
+        C = self.conv_channels
+        b_off = offset + C
+        a_off = b_off + H
+        g_off = a_off + self.decay_rows
         mixed = ctx.buffer("conv_out", (T, C), torch.float32)            # [q | k | v] behind the convolutions
         with ops.section("recurrence.conv"):
-            ops.short_conv(proj[:, offset:offset + C], self.taps, None, tail, ctx.slots, ctx.q_start, mixed, max_new=ctx.max_new)
-            ops.head_unit_norm(mixed, 0, 2 * G, dk, UNIT_EPS, float(dk) ** -0.5, scaled_heads=G)
+            ops.conv_unit_heads(proj[:, offset:offset + C], self.taps, tail, ctx.slots, ctx.q_start, mixed, max_new=ctx.max_new,
+                                heads=2 * G, dim=dk, eps=UNIT_EPS, scale=float(dk) ** -0.5, scaled_heads=G)
         by_channel = self.decay_up is not None
         gate = proj[:, g_off:g_off + self.gate_rows]
         with ops.section("recurrence.gates"):
@@ -162,18 +193,9 @@ class GatedDeltaRule(Part):
             ops.gla_scan(mixed, 0, self.qk, 2 * self.qk, decay, state, ctx.slots, ctx.q_start, raw, num_heads=H,
                          key_dim=dk, value_dim=dv, q_scale=1.0, max_new=ctx.max_new, scratch=ctx.buffer,
                          decay_per_head=not by_channel, qk_heads=G, delta_strength=strength, tensor_cores=rt.fast)
-        o = ctx.buffer("attn_out", (T, self.values), rt.act_dtype)
         with ops.section("recurrence.norm"):
-            clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None
             ops.gla_finish(raw, self.out_gain, s.norm_eps, gate, o, num_heads=H, value_dim=dv, clear=clear,
                            gate_sigmoid=s.gate_activation == "sigmoid")
-        if clear is not None:
-            ctx.note_cleared()
-        with ops.section("recurrence.out"):
-            if overwrite:
-                self.out.store(o, residual, ctx)
-                return False
-            return self.out.accumulate(o, residual, ctx, then_norm)
 
 
 MIXERS.register("gated_delta_rule", GatedDeltaRule)

@@ -262,6 +262,98 @@ def test_an_early_token_comes_through_hundreds_of_steps(products):
     assert float(got[:3].abs().max()) == 0.0
 
 
+# --------------------------------------------------------------------------- what leads up to the recurrence; single steps
+@pytest.mark.parametrize("G,dk,rest,K", [(2, 20, 30, 4), (1, 128, 256, 4), (3, 64, 50, 2), (1, 6, 10, 1), (2, 130, 7, 8), (5, 33, 200, 3), (1, 512, 64, 4)])
+def test_convolutions_with_unit_heads_behind_them(G, dk, rest, K):
+    """Steps of 1, 2, 31, 33 and 100 tokens of two sequences: kept inputs carry over (zeros before the start), queries also
+    times dk^-1/2, the other channels pass unnormed; other slots stay as they were."""
+    from llmplayer_b200.kernels import ops
+    torch.manual_seed(dk + K)
+    C = 2 * G * dk + rest
+    taps = 0.6 * torch.randn(C, K)
+    tail = torch.zeros(4, K - 1, C, device="cuda")
+    tail[1] = 7.0
+    steps = ([1, 2], [33, 1], [2, 100], [100, 31])
+    lengths = [sum(s[i] for s in steps) for i in (0, 1)]
+    xs = [torch.randn(n, C + 9) for n in lengths]
+    refs = []
+    for x in xs:
+        y = P.silu(P.short_convolution(x.double()[:, 4:4 + C], taps.double()))
+        heads = P.unit_length(y[:, :2 * G * dk].reshape(-1, 2 * G, dk))
+        heads[:, :G] *= dk ** -0.5
+        refs.append(torch.cat([heads.reshape(-1, 2 * G * dk), y[:, 2 * G * dk:]], dim=1))
+    done, got = [0, 0], [[], []]
+    for step in steps:
+        x = torch.cat([x[at:at + n] for x, at, n in zip(xs, done, step)]).cuda()
+        out = torch.full((sum(step), C), float("nan"), device="cuda")
+        ops.conv_unit_heads(x[:, 4:4 + C], taps.cuda(), tail, i32([3, 0]), i32([0, step[0], sum(step)]), out, max_new=max(step),
+                            heads=2 * G, dim=dk, eps=1e-6, scale=dk ** -0.5, scaled_heads=G)
+        got[0].append(out[:step[0]].cpu())
+        got[1].append(out[step[0]:].cpu())
+        done = [at + n for at, n in zip(done, step)]
+    for i in (0, 1):
+        check_error("convolutions with unit heads, float32", f"{2 * G} heads of {dk} and {rest} channels, {K} taps, sequence {i}",
+                    rel(torch.cat(got[i]), refs[i]), 5e-6)
+    assert K == 1 or float((tail[1] - 7.0).abs().max()) == 0.0 and float(tail[2].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("low_rank", [True, False])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,dk,dv,ra,rg,K", [(4, 4, 64, 32, 24, 24, 4), (2, 1, 20, 12, 8, 5, 3), (2, 2, 128, 128, 128, 128, 4), (6, 2, 6, 70, 3, 16, 1),
+                                              (1, 1, 256, 40, 40, 8, 2), (2, 1, 130, 300, 16, 24, 8), (1, 1, 300, 10, 7, 7, 4)])
+def test_single_steps_in_one_kernel(H, G, dk, dv, ra, rg, K, dtype, low_rank):
+    """60 steps of one token for three sequences (in slots 4, 0 and 2): projection in, gated heads out, against the plain
+    mechanisms over the whole sequences; both forms of decays and gates; the slots between stay as they were."""
+    from llmplayer_b200.kernels import ops
+    torch.manual_seed(dk + dv)
+    n, B, off = 60, 3, 3
+    C = 2 * G * dk + H * dv
+    rows = (ra, rg) if low_rank else (H, H * dv)
+    F = off + C + H + rows[0] + rows[1] + 2
+    cols = (off, off + C, off + C + H, off + C + H + rows[0])
+    x = torch.randn(B, n, F)
+    taps, gain = 0.6 * torch.randn(C, K), 1 + 0.3 * torch.randn(dv)
+    a_log = torch.randn(H)
+    dt_bias = 1.5 * torch.randn(H * dk if low_rank else H)
+    a_up = (torch.randn(H * dk, ra) / ra ** 0.5).to(dtype) if low_rank else None
+    g_up = (torch.randn(H * dv, rg) / rg ** 0.5).to(dtype) if low_rank else None
+    state, tail = torch.zeros(5, H, dv, dk, device="cuda"), torch.zeros(5, K - 1, C, device="cuda")
+    state[1], tail[3] = 2.0, 5.0
+    slots = i32([4, 0, 2])
+    junk = torch.full((5000,), 3.0, device="cuda")
+    got = []
+    up = {} if not low_rank else {"a_up": a_up.cuda(), "g_up": g_up.cuda()}
+    for t in range(n):
+        out = torch.full((B, H * dv), float("nan"), device="cuda", dtype=dtype)
+        ops.delta_step(x[:, t].contiguous().cuda(), cols, taps.cuda(), tail, state, slots, dt_bias.cuda(), a_log.cuda(), gain.cuda(), 1e-5, out,
+                       num_heads=H, qk_heads=G, key_dim=dk, value_dim=dv, unit_eps=1e-6, q_scale=dk ** -0.5, gate_sigmoid=low_rank, clear=junk, **up)
+        got.append(out.float().cpu())
+    assert float(junk.abs().max()) == 0.0
+    got = torch.stack(got, dim=1)
+    for b in range(B):
+        p = x[b].double()
+        y = P.silu(P.short_convolution(p[:, off:off + C], taps.double()))
+        q = (P.unit_length(y[:, :G * dk].reshape(n, G, dk)) * dk ** -0.5).repeat_interleave(H // G, 1)
+        k = P.unit_length(y[:, G * dk:2 * G * dk].reshape(n, G, dk)).repeat_interleave(H // G, 1)
+        v = y[:, 2 * G * dk:].reshape(n, H, dv)
+        beta = torch.sigmoid(p[:, cols[1]:cols[1] + H])
+        z = p[:, cols[2]:cols[2] + rows[0]]
+        z = (z @ a_up.double().T if low_rank else z) + dt_bias.double()
+        z = P.softplus(z).reshape(n, H, -1)
+        g = torch.exp(-torch.exp(a_log.double())[None, :, None] * z).expand(n, H, dk)
+        o, S = P.channel_delta_recurrence(q, k, v, g, beta)
+        gate = p[:, cols[3]:cols[3] + rows[1]]
+        gate = torch.sigmoid(gate @ g_up.double().T) if low_rank else P.silu(gate)
+        ref = (P.unit_rms(o, 1e-5) * gain.double()).reshape(n, H * dv) * gate
+        # a head whose output nearly cancels is divided by its small root mean square: rounding is amplified there
+        err = ((got[b].double() - ref).abs() / ref.abs().max()).flatten().sort().values
+        assert torch.isfinite(got).all()
+        lim = 1e-4 if dtype == torch.float32 else 5e-3
+        check_error(f"single delta-rule steps, {dtype}", f"{H} heads on {G}, {dk} x {dv}, sequence {b}", float(err[-1]), lim)
+        check_error(f"single delta-rule steps, the state, {dtype}", f"{H} heads on {G}, {dk} x {dv}", rel(state[[4, 0, 2][b]].transpose(1, 2), S), 1e-5)
+    assert float((state[1] - 2.0).abs().max()) == 0.0 and float(state[3].abs().max()) == 0.0 and (K == 1 or float((tail[3] - 5.0).abs().max()) == 0.0)
+
+
 # --------------------------------------------------------------------------- output gate without a gain
 def test_heads_normed_without_a_gain():
     from llmplayer_b200.kernels import ops
