@@ -30,7 +30,8 @@ namespace {
 constexpr int CT = 32;                  // tokens per chunk
 constexpr int HB = 16;                  // tokens per block inside a chunk
 constexpr int NC = 16;                  // value columns per CTA of the second kernel
-constexpr int THREADS = 256;
+constexpr int THREADS = 256;            // of the first kernel
+constexpr int CARRY_THREADS = 512;      // of the second: 16 warps, one per 16 key channels
 constexpr int MAX_DK = 256;
 constexpr size_t MAX_SMEM = 227 * 1024;
 
@@ -297,31 +298,41 @@ __device__ __forceinline__ void cp16(float* dst, const float* src) {
 
 constexpr int SROW = 24;                // floats per row of S and U in shared memory: 16 columns, operand reads without conflicts
 
-// acc[16 x 8] += A[16 x 8 ksteps] X[8 ksteps x 8], A in fragment order, X split into `xh` + `xl` (rows of SROW); three chains
-// of sums
-__device__ __forceinline__ void product(float (*acc)[4], const float* frag, const uint32_t* xh, const uint32_t* xl, int ksteps, int lane) {
+// acc[two tiles of 16 x 8] += A[16 x 8 (s1 - s0)] X[8 (s1 - s0) x 16] for the steps s0 .. s1 - 1 of 8 columns of A (in fragment
+// order), X split into `xh` + `xl` (rows of SROW); three chains of sums per tile
+__device__ __forceinline__ void product(float (*acc)[3][4], const float* frag, const uint32_t* xh, const uint32_t* xl, int s0, int s1,
+                                        int lane) {
     const float4* a = reinterpret_cast<const float4*>(frag) + lane;
     const int at = (lane & 3) * SROW + (lane >> 2);
 #pragma unroll 4
-    for (int s = 0; s < ksteps; ++s) {
+    for (int s = s0; s < s1; ++s) {
         const float4 av = a[s * 32];
-        uint32_t ah[4], al[4], bh[2], bl[2];
-        bh[0] = xh[at + s * 8 * SROW]; bh[1] = xh[at + (s * 8 + 4) * SROW];
-        bl[0] = xl[at + s * 8 * SROW]; bl[1] = xl[at + (s * 8 + 4) * SROW];
+        uint32_t ah[4], al[4];
         split_tf32(av.x, ah[0], al[0]);
         split_tf32(av.y, ah[1], al[1]);
         split_tf32(av.z, ah[2], al[2]);
         split_tf32(av.w, ah[3], al[3]);
-        mma_tf32(acc[0], ah, bh);
-        mma_tf32(acc[1], ah, bl);
-        mma_tf32(acc[2], al, bh);
+#pragma unroll
+        for (int w = 0; w < 2; ++w) {
+            const int e = at + s * 8 * SROW + w * 8;
+            const uint32_t bh[2] = {xh[e], xh[e + 4 * SROW]}, bl[2] = {xl[e], xl[e + 4 * SROW]};
+            mma_tf32(acc[w][0], ah, bh);
+            mma_tf32(acc[w][1], ah, bl);
+            mma_tf32(acc[w][2], al, bh);
+        }
     }
 }
+__device__ __forceinline__ float4 chains(const float (*acc)[4]) {
+    return make_float4(acc[0][0] + (acc[1][0] + acc[2][0]), acc[0][1] + (acc[1][1] + acc[2][1]), acc[0][2] + (acc[1][2] + acc[2][2]),
+                       acc[0][3] + (acc[1][3] + acc[2][3]));
+}
 
-// STAGES: records in flight (two, or one where two do not fit shared memory). TILES: 16 x 8 tiles of the state's columns per
-// warp (dk <= 64 TILES); a warp's threads hold their tiles in registers, shared memory holds the state split for the products.
-template <int STAGES, int TILES>
-__global__ void __launch_bounds__(THREADS)
+// 16 warps. W S and Q S (32 x 16 each) share the warps, four per 16 rows with a quarter of the key channels each (without W,
+// eight per 16 rows of Q S); their parts meet in shared memory. Then warp m owns the state's key channels 16 m .. 16 m + 15:
+// its threads hold those entries in registers, shared memory holds them split for the products.
+// STAGES: records in flight (two, or one where two do not fit shared memory).
+template <int STAGES>
+__global__ void __launch_bounds__(CARRY_THREADS)
 carry_kernel(float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ q_start, int first_chunk, int chunks,
              const float* __restrict__ records, const float* __restrict__ values, float* __restrict__ out, int H, int dk, int dv,
              int delta) {
@@ -331,7 +342,9 @@ carry_kernel(float* __restrict__ state, const int* __restrict__ slots, const int
     uint32_t* Sl = Sh + dkp * SROW;
     uint32_t* Uh = Sl + dkp * SROW;                      // [CT][SROW] twice
     uint32_t* Ul = Uh + CT * SROW;
-    float* ring = reinterpret_cast<float*>(Ul + CT * SROW);      // STAGES records, each followed by the chunk's 32 x 16 values
+    float4* parts = reinterpret_cast<float4*>(Ul + CT * SROW);           // [16 warps][2 tiles][32 lanes]
+    float4* qs = parts + 16 * 64;                                        // [2][2 tiles][32]: Q S
+    float* ring = reinterpret_cast<float*>(qs + 128);    // STAGES records, each followed by the chunk's 32 x 16 values
     const int stage = rec_n + CT * NC;
     lp_grid_release();
     lp_grid_wait();
@@ -348,28 +361,29 @@ carry_kernel(float* __restrict__ state, const int* __restrict__ slots, const int
             const float* src = records + slot * rec_n;
             const float* val = values + slot * value_floats(dv) + blockIdx.x * (CT * NC);
             float* dst = ring + (p % STAGES) * stage;
-            for (int e = tid; e < rec_n / 4; e += THREADS) cp16(dst + 4 * e, src + 4 * e);
-            for (int e = tid; e < CT * NC / 4; e += THREADS) cp16(dst + rec_n + 4 * e, val + 4 * e);
+            for (int e = tid; e < rec_n / 4; e += CARRY_THREADS) cp16(dst + 4 * e, src + 4 * e);
+            for (int e = tid; e < CT * NC / 4; e += CARRY_THREADS) cp16(dst + rec_n + 4 * e, val + 4 * e);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 #pragma unroll
     for (int p = 0; p < STAGES; ++p) request(p);
     const int g8 = lane >> 2, t4 = lane & 3;
-    const int kt = dkp >> 4;
-    // tile `i` of this warp: rows (key channels) 16 m .. of the state, columns 8 w ..
-    float s[TILES][4];
+    const int kt = dkp >> 4, ks = dkp >> 3;
+    const bool owns = warp < kt;
+    float s[2][4];
 #pragma unroll
-    for (int i = 0; i < TILES; ++i) {
-        const int tile = warp + i * (THREADS / 32), m = tile >> 1, w = tile & 1;
+    for (int w = 0; w < 2; ++w)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int r = m * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
-            s[i][e] = (m < kt && j0 + c < dv && r < dk) ? row[(size_t)(j0 + c) * dk + r] : 0.f;
-            if (m < kt) split_tf32(s[i][e], Sh[r * SROW + c], Sl[r * SROW + c]);
+            const int r = warp * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
+            s[w][e] = (owns && j0 + c < dv && r < dk) ? row[(size_t)(j0 + c) * dk + r] : 0.f;
+            if (owns) split_tf32(s[w][e], Sh[r * SROW + c], Sl[r * SROW + c]);
         }
-    }
-    const int role = warp >> 2, mt = (warp >> 1) & 1, nt = warp & 1;       // role 0: W S, then U; role 1: outputs
+    // this warp's share of the first products: rows 16 mt of W (role 0) or Q (role 1), steps s0 .. s1 over the key channels
+    const int nk = delta ? 4 : 8, per = (ks + nk - 1) / nk;
+    const int role = delta ? warp >> 3 : 1, mt = delta ? (warp >> 2) & 1 : warp >> 3;
+    const int s0 = (warp & (nk - 1)) * per, s1 = min(ks, s0 + per);
     for (int p = 0; p < used; ++p) {
         asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 1) : "memory");
         __syncthreads();                            // the record is there, and S as the previous chunk left it
@@ -379,41 +393,61 @@ carry_kernel(float* __restrict__ state, const int* __restrict__ slots, const int
         const float* rec_b = rec_k + CT * dkp;
         const float* rec_p = rec_b + CT * CT;
         const float* val = rec + rec_n;
-        float acc[3][4];
+        {
+            float acc[2][3][4] = {};
+            product(acc, (role == 1 ? rec_q : rec) + mt * ks * 128, Sh, Sl, s0, s1, lane);
+            parts[warp * 64 + lane] = chains(acc[0]);
+            parts[warp * 64 + 32 + lane] = chains(acc[1]);
+        }
+        __syncthreads();
+        if (tid < 256) {                            // thread (product, row half, tile, lane): the parts added, in order
+            const int what = tid >> 7, half = (tid >> 6) & 1, w = (tid >> 5) & 1;
+            float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (what == 1 || delta) {
+                const float4* at = parts + (delta ? what * 8 + half * 4 : half * 8) * 64 + w * 32 + lane;
+                for (int k = 0; k < nk; ++k) {
+                    const float4 v = at[k * 64];
+                    sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
+                }
+            }
+            if (what == 1) qs[half * 64 + w * 32 + lane] = sum;
+            else {
+                const float x[4] = {sum.x, sum.y, sum.z, sum.w};
 #pragma unroll
-        for (int i = 0; i < 3; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-        if (role == 1 || delta)
-            product(acc, (role == 1 ? rec_q : rec) + mt * (dkp >> 3) * 128, Sh + nt * 8, Sl + nt * 8, dkp >> 3, lane);
-        if (role == 0) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = mt * 16 + g8 + (e >> 1) * 8, c = nt * 8 + t4 * 2 + (e & 1);
-                split_tf32(val[r * NC + c] - (acc[0][e] + (acc[1][e] + acc[2][e])), Uh[r * SROW + c], Ul[r * SROW + c]);
+                for (int e = 0; e < 4; ++e) {
+                    const int r = half * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
+                    split_tf32(val[r * NC + c] - x[e], Uh[r * SROW + c], Ul[r * SROW + c]);
+                }
             }
         }
-        __syncthreads();                            // U is there; S has been read
-        if (role == 1) {
-            product(acc, rec_b + mt * (CT >> 3) * 128, Uh + nt * 8, Ul + nt * 8, CT >> 3, lane);
+        __syncthreads();                            // U and Q S are there; S has been read
+        if (owns) {
+            float up[2][3][4] = {};
+            product(up, rec_k + warp * (CT >> 3) * 128, Uh, Ul, 0, CT >> 3, lane);
+            const float p0 = rec_p[warp * 16 + g8], p1 = rec_p[warp * 16 + g8 + 8];
+#pragma unroll
+            for (int w = 0; w < 2; ++w)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int r = warp * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
+                    s[w][e] = fmaf(e < 2 ? p0 : p1, s[w][e], up[w][0][e] + (up[w][1][e] + up[w][2][e]));
+                    split_tf32(s[w][e], Sh[r * SROW + c], Sl[r * SROW + c]);
+                }
+        }
+        if (warp >= 14) {                           // the chunk's outputs: B U joins Q S
+            const int half = warp - 14;
+            float acc[2][3][4] = {};
+            product(acc, rec_b + half * (CT >> 3) * 128, Uh, Ul, 0, CT >> 3, lane);
             const int t = begin + p * CT;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = mt * 16 + g8 + (e >> 1) * 8, c = j0 + nt * 8 + t4 * 2 + (e & 1);
-                if (t + r < t1 && c < dv) out[((size_t)(t + r) * H + h) * dv + c] = acc[0][e] + (acc[1][e] + acc[2][e]);
-            }
-        }
+            for (int w = 0; w < 2; ++w) {
+                const float4 o = qs[half * 64 + w * 32 + lane], u = chains(acc[w]);
+                const float x[4] = {o.x + u.x, o.y + u.y, o.z + u.z, o.w + u.w};
 #pragma unroll
-        for (int i = 0; i < TILES; ++i) {
-            const int tile = warp + i * (THREADS / 32), m = tile >> 1, w = tile & 1;
-            if (m >= kt) break;
-            float up[3][4];
-#pragma unroll
-            for (int e = 0; e < 3; ++e) up[e][0] = up[e][1] = up[e][2] = up[e][3] = 0.f;
-            product(up, rec_k + m * (CT >> 3) * 128, Uh + w * 8, Ul + w * 8, CT >> 3, lane);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int r = m * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
-                s[i][e] = fmaf(rec_p[r], s[i][e], up[0][e] + (up[1][e] + up[2][e]));
-                split_tf32(s[i][e], Sh[r * SROW + c], Sl[r * SROW + c]);
+                for (int e = 0; e < 4; ++e) {
+                    const int r = half * 16 + g8 + (e >> 1) * 8, c = j0 + w * 8 + t4 * 2 + (e & 1);
+                    if (t + r < t1 && c < dv) out[((size_t)(t + r) * H + h) * dv + c] = x[e];
+                }
             }
         }
         __syncthreads();                            // the stage is free
@@ -421,14 +455,12 @@ carry_kernel(float* __restrict__ state, const int* __restrict__ slots, const int
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
-    for (int i = 0; i < TILES; ++i) {
-        const int tile = warp + i * (THREADS / 32), m = tile >> 1, w = tile & 1;
+    for (int w = 0; w < 2; ++w)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int r = m * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
-            if (m < kt && j0 + c < dv && r < dk) row[(size_t)(j0 + c) * dk + r] = s[i][e];
+            const int r = warp * 16 + g8 + (e >> 1) * 8, c = w * 8 + t4 * 2 + (e & 1);
+            if (owns && j0 + c < dv && r < dk) row[(size_t)(j0 + c) * dk + r] = s[w][e];
         }
-    }
 }
 
 template <typename K> int reserve(K kernel, size_t bytes, size_t& granted) {
@@ -469,17 +501,16 @@ extern "C" int lp_chunked_recurrence(const float* proj, int ld, int q_off, int k
     const int dkp = padded(dk), delta = beta ? 1 : 0;
     const size_t smem_p = ((size_t)(3 * CT + 3 * HB) * (dkp + 4) + 2 * CT * CT + CT) * sizeof(float);
     const size_t stage = (size_t)(record_floats(dkp, delta) + CT * NC) * sizeof(float);
-    const size_t kept = (size_t)(dkp + CT) * SROW * 2 * sizeof(float);
+    const size_t kept = (size_t)(dkp + CT) * SROW * 2 * sizeof(float) + (16 * 64 + 128) * sizeof(float4);
     const bool two = kept + 2 * stage <= MAX_SMEM;
     const size_t smem_c = kept + (two ? 2 : 1) * stage;
     auto prepare = dk <= 64 ? prepare_kernel<4> : dk <= 128 ? prepare_kernel<8> : prepare_kernel<16>;
     const int size = dk <= 64 ? 0 : dk <= 128 ? 1 : 2;
-    auto carry = two ? (size == 0 ? carry_kernel<2, 1> : size == 1 ? carry_kernel<2, 2> : carry_kernel<2, 4>)
-                     : (size == 0 ? carry_kernel<1, 1> : size == 1 ? carry_kernel<1, 2> : carry_kernel<1, 4>);
-    static size_t granted_p[3] = {}, granted_c[2][3] = {};       // what each kernel has been allowed so far
+    auto carry = two ? carry_kernel<2> : carry_kernel<1>;
+    static size_t granted_p[3] = {}, granted_c[2] = {};       // what each kernel has been allowed so far
     int rc = reserve(prepare, smem_p, granted_p[size]);
     if (rc) return rc;
-    rc = reserve(carry, smem_c, granted_c[two ? 1 : 0][size]);
+    rc = reserve(carry, smem_c, granted_c[two ? 1 : 0]);
     if (rc) return rc;
     const int total = (max_new + CT - 1) / CT;
     for (int first = 0; first < total; first += chunks) {
@@ -487,7 +518,7 @@ extern "C" int lp_chunked_recurrence(const float* proj, int ld, int q_off, int k
         lp_launch(prepare, dim3(here, H, B), THREADS, smem_p, stream, in, q_start, first, chunks, records, values);
         rc = lp_check_launch("chunked_recurrence (prepare)");
         if (rc) return rc;
-        lp_launch(carry, dim3((dv + NC - 1) / NC, H, B), THREADS, smem_c, stream, state, slots, q_start, first, chunks,
+        lp_launch(carry, dim3((dv + NC - 1) / NC, H, B), CARRY_THREADS, smem_c, stream, state, slots, q_start, first, chunks,
                   (const float*)records, (const float*)values, out, H, dk, dv, delta);
         rc = lp_check_launch("chunked_recurrence (carry)");
         if (rc) return rc;
