@@ -146,8 +146,10 @@ prepare_kernel(Inputs in, const int* __restrict__ q_start, int first_chunk, int 
     for (int e = tid; e < CT * CT; e += THREADS) L[e] = Bm[e] = 0.f;
     __syncthreads();
 
-    // products of decays, a thread per key channel; its column of diag(b) (P k) stays in registers for the solve
+    // products of decays, a thread per key channel (forwards; its column of diag(b) (P k) stays in registers for the solve) and
+    // one backwards (other threads where there are enough)
     float col[CT];
+    const int back = dkp <= THREADS / 2 ? THREADS / 2 : 0;
     if (tid < dkp) {
         const int c = tid;
         float p = 1.f, pb = 1.f;
@@ -164,8 +166,10 @@ prepare_kernel(Inputs in, const int* __restrict__ q_start, int first_chunk, int 
             }
         }
         rec_p[c] = p;
-        p = 1.f;
-        pb = 1.f;
+    }
+    if (tid >= back && tid - back < dkp) {
+        const int c = tid - back;
+        float p = 1.f, pb = 1.f;
 #pragma unroll
         for (int i = CT - 1; i >= 0; --i) {
             const float g = gs[i * ks + c], k = kk[i * ks + c];

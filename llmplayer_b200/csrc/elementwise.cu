@@ -1079,7 +1079,8 @@ extern "C" int lp_scaled_sum(float* x, const float* a, const float* va, float sa
 // fixed order. The new row lies in shared memory (d floats) so that warps can take the sums of the parts whatever their
 // borders: every part is cut into `cuts` slices, a warp sums a slice, a part's slices are added in order.
 constexpr int PAIR_NORM_MAX_SLICES = 1024;
-template <typename TOut>
+constexpr int PAIR_NORM_QUADS = 4;           // float4 per thread and operand: rows up to 256 * 4 * 4 = 4096 values
+template <typename TOut, bool VEC>
 __global__ void __launch_bounds__(NORM_THREADS)
 pair_norm_add_kernel(const float* __restrict__ a, const float* __restrict__ wa, float sa, float eps_a,
                      const float* __restrict__ b, const float* __restrict__ wb, float sb, float eps_b, float* __restrict__ x,
@@ -1096,18 +1097,55 @@ pair_norm_add_kernel(const float* __restrict__ a, const float* __restrict__ wa, 
     const float* br = b + row * d;
     float* xr = x + row * d;
     float s0 = 0.f, s1 = 0.f;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        const float u = ar[i], v = br[i];
-        s0 += u * u;
-        s1 += v * v;
-    }
-    s0 = lp_block_sum(s0, scratch);
-    s1 = lp_block_sum(s1, scratch);
-    const float fa = sa / sqrtf(s0 / (float)d + eps_a), fb = sb / sqrtf(s1 / (float)d + eps_b);
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        const float v = xr[i] + (ar[i] * fa * wa[i] + br[i] * fb * wb[i]);
-        xr[i] = v;
-        sum_row[i] = v;
+    if (VEC) {
+        // four values per load, a row's values kept in registers between the two passes
+        float4 u[PAIR_NORM_QUADS], v[PAIR_NORM_QUADS], r[PAIR_NORM_QUADS];
+        const int quads = d >> 2;
+#pragma unroll
+        for (int k = 0; k < PAIR_NORM_QUADS; ++k) {
+            const int i = threadIdx.x + k * NORM_THREADS;
+            u[k] = v[k] = r[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < quads) {
+                u[k] = reinterpret_cast<const float4*>(ar)[i];
+                v[k] = reinterpret_cast<const float4*>(br)[i];
+                r[k] = reinterpret_cast<const float4*>(xr)[i];
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < PAIR_NORM_QUADS; ++k) {
+            s0 += (u[k].x * u[k].x + u[k].y * u[k].y) + (u[k].z * u[k].z + u[k].w * u[k].w);
+            s1 += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+        }
+        s0 = lp_block_sum(s0, scratch);
+        s1 = lp_block_sum(s1, scratch);
+        const float fa = sa / sqrtf(s0 / (float)d + eps_a), fb = sb / sqrtf(s1 / (float)d + eps_b);
+#pragma unroll
+        for (int k = 0; k < PAIR_NORM_QUADS; ++k) {
+            const int i = threadIdx.x + k * NORM_THREADS;
+            if (i < quads) {
+                const float4 ga = reinterpret_cast<const float4*>(wa)[i], gb = reinterpret_cast<const float4*>(wb)[i];
+                r[k].x += u[k].x * fa * ga.x + v[k].x * fb * gb.x;
+                r[k].y += u[k].y * fa * ga.y + v[k].y * fb * gb.y;
+                r[k].z += u[k].z * fa * ga.z + v[k].z * fb * gb.z;
+                r[k].w += u[k].w * fa * ga.w + v[k].w * fb * gb.w;
+                reinterpret_cast<float4*>(xr)[i] = r[k];
+                reinterpret_cast<float4*>(sum_row)[i] = r[k];
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            const float u = ar[i], v = br[i];
+            s0 += u * u;
+            s1 += v * v;
+        }
+        s0 = lp_block_sum(s0, scratch);
+        s1 = lp_block_sum(s1, scratch);
+        const float fa = sa / sqrtf(s0 / (float)d + eps_a), fb = sb / sqrtf(s1 / (float)d + eps_b);
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            const float v = xr[i] + (ar[i] * fa * wa[i] + br[i] * fb * wb[i]);
+            xr[i] = v;
+            sum_row[i] = v;
+        }
     }
     if (!w2) return;
     __syncthreads();
@@ -1116,6 +1154,7 @@ pair_norm_add_kernel(const float* __restrict__ a, const float* __restrict__ wa, 
     for (int k = warp; k < parts * cuts; k += NORM_THREADS / 32) {
         const int p = k / cuts, lo = (k - p * cuts) * piece, hi = min(width, lo + piece);
         float ss = 0.f;
+#pragma unroll 4
         for (int i = lo + lane; i < hi; i += 32) {
             const float v = sum_row[p * width + i];
             ss += v * v;
@@ -1125,6 +1164,17 @@ pair_norm_add_kernel(const float* __restrict__ a, const float* __restrict__ wa, 
     }
     __syncthreads();
     TOut* o = out2 + row * d;
+    if (VEC && (width & 3) == 0) {
+        for (int q = threadIdx.x; q < d >> 2; q += NORM_THREADS) {
+            const int p = 4 * q / width;
+            float ss = 0.f;
+            for (int c = 0; c < cuts; ++c) ss += slice[p * cuts + c];
+            const float f = 1.0f / sqrtf(ss / (float)width + eps2);
+            const float4 v = reinterpret_cast<const float4*>(sum_row)[q], g = reinterpret_cast<const float4*>(w2)[q];
+            store4<TOut>(o + 4 * q, v.x * f * g.x, v.y * f * g.y, v.z * f * g.z, v.w * f * g.w);
+        }
+        return;
+    }
     int held = -1;
     float f = 0.f;
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
@@ -1148,13 +1198,20 @@ extern "C" int lp_pair_norm_add(const float* a, const float* wa, float sa, float
     const int cuts = parts >= NORM_THREADS / 32 ? 1 : (NORM_THREADS / 32 + parts - 1) / parts;
     const size_t smem = (size_t)d * sizeof(float);
     if (smem > 200 * 1024) LP_REFUSE("pair_norm_add: rows of %d values do not fit shared memory", d);
+    const bool vec = d % 4 == 0 && d <= NORM_THREADS * 4 * PAIR_NORM_QUADS &&
+                     (((uintptr_t)a | (uintptr_t)b | (uintptr_t)x | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)w2 | (uintptr_t)out2) & 15) == 0;
 #define LP_LAUNCH_PAIR_NORM(TOUT)                                                                                          \
     do {                                                                                                                   \
+        if (vec) {                                                                                                         \
+            lp_launch(pair_norm_add_kernel<TOUT, true>, T, NORM_THREADS, smem, stream, a, wa, sa, eps_a, b, wb, sb, eps_b, x, w2, eps2, \
+                      parts, cuts, (TOUT*)out2, d, zero, zero_count);                                                      \
+            break;                                                                                                         \
+        }                                                                                                                  \
         if (smem > 40 * 1024) {                                                                                            \
-            cudaError_t e = cudaFuncSetAttribute(pair_norm_add_kernel<TOUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(pair_norm_add_kernel<TOUT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) LP_REFUSE("pair_norm_add: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e)); \
         }                                                                                                                  \
-        lp_launch(pair_norm_add_kernel<TOUT>, T, NORM_THREADS, smem, stream, a, wa, sa, eps_a, b, wb, sb, eps_b, x, w2, eps2, parts, \
+        lp_launch(pair_norm_add_kernel<TOUT, false>, T, NORM_THREADS, smem, stream, a, wa, sa, eps_a, b, wb, sb, eps_b, x, w2, eps2, parts, \
                   cuts, (TOUT*)out2, d, zero, zero_count);                                                                 \
     } while (0)
     if (!out2 || out2_dtype == LP_F32) LP_LAUNCH_PAIR_NORM(float);

@@ -588,6 +588,8 @@ short_conv_kernel(const float* __restrict__ in, int ldi, const TW* __restrict__ 
 // eps), the first `scaled` heads also times `scale`). A block takes whole heads (`per_block` of them, `head_warps` warps each)
 // or, behind them, as many single channels as it has threads; a thread keeps its channel's 32 outputs in registers, and a
 // warp's sums over its channels meet in a transposing reduction that leaves token t's sum in lane t.
+// TAPS: the most taps (K of them are used).
+template <int TAPS>
 __global__ void __launch_bounds__(512)
 conv_unit_heads_kernel(const float* __restrict__ in, int ldi, const float* __restrict__ taps, float* __restrict__ tail,
                        const int* __restrict__ slots, const int* __restrict__ q_start, float* __restrict__ out, int ldo, int C, int K,
@@ -610,21 +612,21 @@ conv_unit_heads_kernel(const float* __restrict__ in, int ldi, const float* __res
 #pragma unroll
     for (int i = 0; i < CONV_CHUNK; ++i) y[i] = 0.f;
     if (valid) {
-        float w[CONV_MAX_TAPS], hist[CONV_MAX_TAPS - 1];
+        float w[TAPS], hist[TAPS - 1];
 #pragma unroll
-        for (int j = 0; j < CONV_MAX_TAPS; ++j) {
-            const int tap = j - (CONV_MAX_TAPS - K);
+        for (int j = 0; j < TAPS; ++j) {
+            const int tap = j - (TAPS - K);
             w[j] = tap >= 0 ? taps[(long long)c * K + tap] : 0.f;
         }
         float* keep = tail + (long long)slots[b] * (K - 1) * C + c;
 #pragma unroll
-        for (int i = 0; i < CONV_MAX_TAPS - 1; ++i) {
+        for (int i = 0; i < TAPS - 1; ++i) {
             float v = 0.f;
             if (i < K - 1) {
                 const int src = begin - 1 - i;
                 v = src >= t0 ? in[(long long)src * ldi + c] : keep[(long long)(K - 1 + src - t0) * C];
             }
-            hist[CONV_MAX_TAPS - 2 - i] = v;
+            hist[TAPS - 2 - i] = v;
         }
         if (begin == t0) {                                      // the step's last K - 1 inputs become the tail, as above
             for (int j = 0; j < K - 1; ++j) {
@@ -639,11 +641,11 @@ conv_unit_heads_kernel(const float* __restrict__ in, int ldi, const float* __res
         for (int i = 0; i < CONV_CHUNK; ++i) {
             float acc = 0.f;
 #pragma unroll
-            for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) {
-                const int at = i - (CONV_MAX_TAPS - 1) + j;     // the input 7 - j tokens back
-                acc = fmaf(w[j], at >= 0 ? x[at >= 0 ? at : 0] : hist[at + CONV_MAX_TAPS - 1 < CONV_MAX_TAPS - 1 ? at + CONV_MAX_TAPS - 1 : 0], acc);
+            for (int j = 0; j < TAPS - 1; ++j) {
+                const int at = i - (TAPS - 1) + j;     // the input 7 - j tokens back
+                acc = fmaf(w[j], at >= 0 ? x[at >= 0 ? at : 0] : hist[at + TAPS - 1 < TAPS - 1 ? at + TAPS - 1 : 0], acc);
             }
-            acc = fmaf(w[CONV_MAX_TAPS - 1], x[i], acc);
+            acc = fmaf(w[TAPS - 1], x[i], acc);
             y[i] = i < n ? acc / (1.0f + expf(-acc)) : 0.f;
         }
     }
@@ -714,7 +716,7 @@ struct RankMap {
 };
 constexpr int RM_TOKENS = 128, RM_TILE = 64, RM_K = 32;
 
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 low_rank_gates_kernel(const float* __restrict__ proj, int ld, int T, int H, RankMap a, const float* __restrict__ dt_bias,
                       const float* __restrict__ a_log, int dk, RankMap g, int a_tiles, int b_off, float* __restrict__ strength) {
     __shared__ float low[RM_K][RM_TOKENS + 4], up[RM_K][RM_TILE + 4];
@@ -730,28 +732,41 @@ low_rank_gates_kernel(const float* __restrict__ proj, int ld, int T, int H, Rank
     for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    const int lr = threadIdx.x % RM_K, li = threadIdx.x / RM_K;          // a thread loads column lr of every eighth row
+    // a thread loads columns lr, lr + 8, ... of rows li, li + 4, ... of its warp's share: whole sectors from memory, and the
+    // transposing stores of a warp fall into 32 different banks; the next columns are on their way during the sums
+    const int lr = threadIdx.x & 7, li = (threadIdx.x >> 3) & 3, warp = threadIdx.x >> 5;
+    float x[4][4], w[4][2];
+    auto load = [&](int r0) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int r = r0 + lr + 8 * k;
+            const bool in = r < m.rank;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int t = t0 + warp * 16 + li + 4 * u;
+                x[k][u] = (in && t < T) ? __ldg(proj + (long long)t * ld + m.off + r) : 0.f;
+            }
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int c = c0 + warp * 8 + li + 4 * u;
+                const long long at = (long long)c * m.rank + r;
+                w[k][u] = 0.f;
+                if (in && c < m.channels) w[k][u] = m.up_bf16 ? __bfloat162float(((const __nv_bfloat16*)m.up)[at]) : ((const float*)m.up)[at];
+            }
+        }
+    };
+    load(0);
     for (int r0 = 0; r0 < m.rank; r0 += RM_K) {
-        const bool in = r0 + lr < m.rank;
-        float x[RM_TOKENS / 8], w[RM_TILE / 8];
-#pragma unroll
-        for (int u = 0; u < RM_TOKENS / 8; ++u) {
-            const int t = t0 + li + 8 * u;
-            x[u] = (in && t < T) ? __ldg(proj + (long long)t * ld + m.off + r0 + lr) : 0.f;
-        }
-#pragma unroll
-        for (int u = 0; u < RM_TILE / 8; ++u) {
-            const int c = c0 + li + 8 * u;
-            const long long at = (long long)c * m.rank + r0 + lr;
-            w[u] = 0.f;
-            if (in && c < m.channels) w[u] = m.up_bf16 ? __bfloat162float(((const __nv_bfloat16*)m.up)[at]) : ((const float*)m.up)[at];
-        }
         __syncthreads();
 #pragma unroll
-        for (int u = 0; u < RM_TOKENS / 8; ++u) low[lr][li + 8 * u] = x[u];
+        for (int k = 0; k < 4; ++k) {
 #pragma unroll
-        for (int u = 0; u < RM_TILE / 8; ++u) up[lr][li + 8 * u] = w[u];
+            for (int u = 0; u < 4; ++u) low[lr + 8 * k][warp * 16 + li + 4 * u] = x[k][u];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) up[lr + 8 * k][warp * 8 + li + 4 * u] = w[k][u];
+        }
         __syncthreads();
+        if (r0 + RM_K < m.rank) load(r0 + RM_K);
 #pragma unroll 8
         for (int r = 0; r < RM_K; ++r) {
             const float4 xa = *reinterpret_cast<const float4*>(&low[r][ty * 8]), xb = *reinterpret_cast<const float4*>(&low[r][ty * 8 + 4]);
@@ -1029,8 +1044,8 @@ extern "C" int lp_conv_unit_heads(const float* in, int ldi, const float* taps, f
     const int head_warps = (dim + 31) / 32, per_block = head_warps >= 4 ? 1 : 4 / head_warps;
     const int threads = head_warps * per_block * 32;
     const int head_blocks = (heads + per_block - 1) / per_block, rest = (C - heads * dim + threads - 1) / threads;
-    lp_launch(conv_unit_heads_kernel, dim3(head_blocks + rest, chunks, B), threads, 0, stream, in, ldi, taps, tail, slots, q_start, out, ldo,
-              C, K, heads, dim, head_warps, per_block, head_blocks, eps, scale, scaled);
+    lp_launch(K <= 4 ? conv_unit_heads_kernel<4> : conv_unit_heads_kernel<CONV_MAX_TAPS>, dim3(head_blocks + rest, chunks, B), threads, 0,
+              stream, in, ldi, taps, tail, slots, q_start, out, ldo, C, K, heads, dim, head_warps, per_block, head_blocks, eps, scale, scaled);
     return lp_check_launch("conv_unit_heads");
 }
 
