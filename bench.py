@@ -527,7 +527,7 @@ def dopuvik_rooflines(size, layers, row, peaks, batch, context, n):
         "decode dopuvik attention with kept tokens (of copy bandwidth)": frac(
             batch * min(context, W + K) * 2 * G * hd * 2, dec.get("left.attention.scores"), n_pair, gbs),
         "decode dopuvik state-space recurrence (of copy bandwidth)": frac(batch * sh * sn * sp * 4 * 2, dec.get("recurrence.scan"), n_space, gbs),
-        "decode dopuvik delta-rule recurrence (of copy bandwidth)": frac(batch * gh * gk * gk * 4 * 2, dec.get("right.recurrence.scan"), n_pair, gbs),
+        "decode dopuvik delta-rule recurrence (of copy bandwidth)": frac(batch * gh * gk * gk * 4 * 2, dec.get("right.recurrence.step"), n_pair, gbs),
     }
     if z is not None:
         zh, zn = width // 64, 64
@@ -577,7 +577,7 @@ def vomotar_rooflines(size, layers, row, peaks, batch, context, n):
             batch * (context % W) * 2 * G * hd * 2, dec.get("left.attention.scores"), n_pair, gbs),
         "decode vomotar retention recurrence (of copy bandwidth)": frac(batch * gh * gk * gv * 4 * 2, dec.get("right.recurrence.scan"), n_pair, gbs),
         "decode vomotar delta-rule recurrence (of copy bandwidth)": frac(
-            batch * gh * gk * gk * 4 * 2, dec.get("recurrence.scan", dec.get("recurrence.step")), n_delta, gbs),
+            batch * gh * gk * gk * 4 * 2, dec.get("recurrence.step"), n_delta, gbs),
     }
 
 
