@@ -575,7 +575,7 @@ def vomotar_rooflines(size, layers, row, peaks, batch, context, n):
         "prefill vomotar two normed results summed (of copy bandwidth)": frac(n * width * (4 * 4 + 2), pre.get("mixer.sum"), n_pair, gbs),
         "decode vomotar attention in chunks (of copy bandwidth)": frac(
             batch * (context % W) * 2 * G * hd * 2, dec.get("left.attention.scores"), n_pair, gbs),
-        "decode vomotar retention recurrence (of copy bandwidth)": frac(batch * gh * gk * gv * 4 * 2, dec.get("right.recurrence.scan"), n_pair, gbs),
+        "decode vomotar retention recurrence (of copy bandwidth)": frac(batch * gh * gk * gv * 4 * 2, dec.get("right.recurrence.step"), n_pair, gbs),
         "decode vomotar delta-rule recurrence (of copy bandwidth)": frac(
             batch * gh * gk * gk * 4 * 2, dec.get("recurrence.step"), n_delta, gbs),
     }

@@ -1,5 +1,5 @@
-// One token per sequence through a delta-rule layer, from the projection of the layer's input to the input of its output
-// product, in one kernel (the single steps of linear_attention.cu, fused for decode steps):
+// One token per sequence through a recurrent layer, from the projection of the layer's input to the input of its output
+// product, in one kernel (the single steps of linear_attention.cu, fused for decode steps). The delta rule:
 //
 //   short convolutions of the query, key and value channels (the kept inputs move on), silu, unit queries and keys, write
 //   strength, decays (one per head, or one per head and key channel from a low-rank map), S <- a S; u = b (v - S^T k);
@@ -9,7 +9,9 @@
 // One CTA per (query / key head, sequence): it forms the head's query and key once and serves every value head that reads
 // them, so nothing that one CTA renews (state, kept inputs) is read by another. 16 lanes share a value column's key
 // channels (four neighbouring channels per lane and load); the read-outs S^T k and S^T q of a column meet in four shuffles
-// and come from the decayed state before the write: o = S^T q + u (k . q). All arithmetic is float32.
+// and come from the decayed state before the write: o = S^T q + u (k . q). Retention: queries and keys rotated by their
+// position, S <- d S + k v^T with a constant d per head, o = S^T q, the norm of the head's o without a gain, the silu gate; a
+// CTA per head and sequence. All arithmetic is float32.
 #include "common.cuh"
 
 namespace {
@@ -96,6 +98,48 @@ __device__ __forceinline__ float quarter_dot(const TW* up, const float* low, int
     return acc;
 }
 
+// The state entries of the lane's channels 64 u + 4 l16 + e of JT neighbouring columns from column j0 on.
+template <int KPT, int JT>
+__device__ __forceinline__ void load_columns(float (*s)[KPT], const float* S, int j0, int l16, int dk, int dv) {
+    const bool quads = (dk & 3) == 0;
+#pragma unroll
+    for (int jj = 0; jj < JT; ++jj) {
+        const int j = j0 + jj;
+#pragma unroll
+        for (int u = 0; u < KPT / 4; ++u) {
+            const int c = 64 * u + 4 * l16;
+            if (quads) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (j < dv && c < dk) v = *reinterpret_cast<const float4*>(S + (size_t)j * dk + c);
+                s[jj][4 * u] = v.x; s[jj][4 * u + 1] = v.y; s[jj][4 * u + 2] = v.z; s[jj][4 * u + 3] = v.w;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[jj][4 * u + e] = (j < dv && c + e < dk) ? S[(size_t)j * dk + c + e] : 0.f;
+            }
+        }
+    }
+}
+template <int KPT, int JT>
+__device__ __forceinline__ void store_columns(const float (*s)[KPT], float* S, int j0, int l16, int dk, int dv) {
+    const bool quads = (dk & 3) == 0;
+#pragma unroll
+    for (int jj = 0; jj < JT; ++jj) {
+        const int j = j0 + jj;
+#pragma unroll
+        for (int u = 0; u < KPT / 4; ++u) {
+            const int c = 64 * u + 4 * l16;
+            if (j >= dv || c >= dk) continue;
+            if (quads)
+                *reinterpret_cast<float4*>(S + (size_t)j * dk + c) = make_float4(s[jj][4 * u], s[jj][4 * u + 1], s[jj][4 * u + 2], s[jj][4 * u + 3]);
+            else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (c + e < dk) S[(size_t)j * dk + c + e] = s[jj][4 * u + e];
+            }
+        }
+    }
+}
+
 // TW: number format of the low-rank maps. KPT: key channels per lane (dk <= 16 KPT), JT: neighbouring value columns per 16 lanes.
 template <typename TW, int KPT, int JT, typename TOut>
 __global__ void __launch_bounds__(THREADS)
@@ -118,28 +162,10 @@ delta_step_kernel(const StepArgs a, TOut* __restrict__ out) {
     const int qk = a.G * dk, channels = 2 * qk + a.H * dv;
     float* kept = a.tail + (size_t)a.slots[b] * (a.K - 1) * channels;
     const int l16 = tid & 15, grp = tid >> 4;
-    const bool quads = (dk & 3) == 0;
 
-    // the state entries of the lane's channels 64 u + 4 l16 + e of JT columns, requested ahead of what they meet
-    float s[JT][KPT];
+    float s[JT][KPT];                   // requested ahead of what they meet
     auto load = [&](int h, int base) {
-        const float* S = a.state + ((size_t)a.slots[b] * a.H + h) * dv * dk;
-#pragma unroll
-        for (int jj = 0; jj < JT; ++jj) {
-            const int j = base + grp * JT + jj;
-#pragma unroll
-            for (int u = 0; u < KPT / 4; ++u) {
-                const int c = 64 * u + 4 * l16;
-                if (quads) {
-                    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (j < dv && c < dk) v = *reinterpret_cast<const float4*>(S + (size_t)j * dk + c);
-                    s[jj][4 * u] = v.x; s[jj][4 * u + 1] = v.y; s[jj][4 * u + 2] = v.z; s[jj][4 * u + 3] = v.w;
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) s[jj][4 * u + e] = (j < dv && c + e < dk) ? S[(size_t)j * dk + c + e] : 0.f;
-                }
-            }
-        }
+        load_columns<KPT, JT>(s, a.state + ((size_t)a.slots[b] * a.H + h) * dv * dk, base + grp * JT, l16, dk, dv);
     };
     load(g * R, 0);
     if (a.a_up)
@@ -232,23 +258,7 @@ delta_step_kernel(const StepArgs a, TOut* __restrict__ out) {
 #pragma unroll
                 for (int jj = 0; jj < JT; ++jj) s[jj][u] = fmaf(k, r1[jj], s[jj][u]);
             }
-#pragma unroll
-            for (int jj = 0; jj < JT; ++jj) {
-                const int j = base + grp * JT + jj;
-#pragma unroll
-                for (int u = 0; u < KPT / 4; ++u) {
-                    const int c = 64 * u + 4 * l16;
-                    if (j >= dv || c >= dk) continue;
-                    if (quads)
-                        *reinterpret_cast<float4*>(S + (size_t)j * dk + c) =
-                            make_float4(s[jj][4 * u], s[jj][4 * u + 1], s[jj][4 * u + 2], s[jj][4 * u + 3]);
-                    else {
-#pragma unroll
-                        for (int e = 0; e < 4; ++e)
-                            if (c + e < dk) S[(size_t)j * dk + c + e] = s[jj][4 * u + e];
-                    }
-                }
-            }
+            store_columns<KPT, JT>(s, S, base + grp * JT, l16, dk, dv);
             if (base + GROUPS * JT < dv) load(h, base + GROUPS * JT);
             else if (r + 1 < R) load(h + 1, 0);
         }
@@ -266,9 +276,132 @@ delta_step_kernel(const StepArgs a, TOut* __restrict__ out) {
     }
 }
 
+
+// ---------------------------------------------------------------- retention
+struct RetentionArgs {
+    const float* proj;         // [B, ld]: queries, keys [H, dk], values, gate [H, dv]
+    int ld, q_off, k_off, v_off, g_off;
+    const float* inv_freq;     // [rd / 2] or null
+    int rd, interleaved;
+    const int* positions;      // [B]
+    const float* decays;       // [H]
+    float q_scale, norm_eps;
+    float* state;              // [slots, H, dv, dk]
+    const int* slots;
+    int H, dk, dv;
+    float* zero;
+    long long zero_count;
+};
+
+template <int KPT, int JT, typename TOut>
+__global__ void __launch_bounds__(THREADS)
+retention_step_kernel(const RetentionArgs a, TOut* __restrict__ out) {
+    extern __shared__ float sm[];
+    const int dk = a.dk, dv = a.dv;
+    float* q_s = sm;                    // [dk]
+    float* k_s = q_s + dk;              // [dk]
+    float* v_s = k_s + dk;              // [dv]
+    float* o_s = v_s + dv;              // [dv]
+    const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+    lp_grid_release();
+    lp_grid_wait();
+    clear_on_the_side(a.zero, a.zero_count);
+    const int l16 = tid & 15, grp = tid >> 4;
+    const float* row = a.proj + (size_t)b * a.ld;
+    float* S = a.state + ((size_t)a.slots[b] * a.H + h) * dv * dk;
+    float s[JT][KPT];
+    load_columns<KPT, JT>(s, S, grp * JT, l16, dk, dv);
+    for (int i = tid; i < 2 * dk; i += THREADS) {
+        const int c = i < dk ? i : i - dk;
+        const float* head = row + (i < dk ? a.q_off : a.k_off) + h * dk;
+        float val = head[c];
+        if (c < a.rd) {
+            const int half = a.rd >> 1;
+            const bool first = a.interleaved ? (c & 1) == 0 : c < half;
+            const int pair = a.interleaved ? c >> 1 : (first ? c : c - half);
+            const float other = head[a.interleaved ? (c ^ 1) : (first ? c + half : c - half)];
+            float sn, cs;
+            sincosf((float)a.positions[b] * a.inv_freq[pair], &sn, &cs);
+            val = first ? val * cs - other * sn : val * cs + other * sn;
+        }
+        (i < dk ? q_s : k_s)[c] = i < dk ? val * a.q_scale : val;
+    }
+    for (int j = tid; j < dv; j += THREADS) v_s[j] = row[a.v_off + h * dv + j];
+    __syncthreads();
+    const float d = a.decays[h];
+    for (int base = 0; base < dv; base += GROUPS * JT) {
+        const int j0 = base + grp * JT;
+        float v[JT], r[JT];
+#pragma unroll
+        for (int jj = 0; jj < JT; ++jj) {
+            v[jj] = j0 + jj < dv ? v_s[j0 + jj] : 0.f;
+            r[jj] = 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < KPT; ++u) {
+            const int c = 64 * (u >> 2) + 4 * l16 + (u & 3);
+            const float k = c < dk ? k_s[c] : 0.f, q = c < dk ? q_s[c] : 0.f;
+#pragma unroll
+            for (int jj = 0; jj < JT; ++jj) {
+                s[jj][u] = fmaf(d, s[jj][u], k * v[jj]);
+                r[jj] = fmaf(s[jj][u], q, r[jj]);
+            }
+        }
+        store_columns<KPT, JT>(s, S, j0, l16, dk, dv);
+        if (base + GROUPS * JT < dv) load_columns<KPT, JT>(s, S, j0 + GROUPS * JT, l16, dk, dv);
+#pragma unroll
+        for (int o = 1; o < 16; o <<= 1)
+#pragma unroll
+            for (int jj = 0; jj < JT; ++jj) r[jj] += __shfl_xor_sync(0xffffffffu, r[jj], o);
+#pragma unroll
+        for (int jj = 0; jj < JT; ++jj)
+            if (l16 == 0 && j0 + jj < dv) o_s[j0 + jj] = r[jj];
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int j = lane; j < dv; j += 32) ss = fmaf(o_s[j], o_s[j], ss);
+    ss = lp_warp_sum(ss);
+    const float f = 1.0f / sqrtf(ss / (float)dv + a.norm_eps);
+    for (int j = tid; j < dv; j += THREADS) {
+        const float z = row[a.g_off + h * dv + j];
+        out[((size_t)b * a.H + h) * dv + j] = lp_from_float<TOut>(o_s[j] * f * (z * sigmoid(z)));
+    }
+}
+
 }  // namespace
 
-// One new token for each of B sequences. proj: float32 [B, ld] (see StepArgs for the columns); out: [B, H * dv] float32 or
+// One new token for each of B sequences through a retention. proj: float32 [B, ld] (see RetentionArgs for the columns); positions:
+// int32 [B]; out: [B, H * dv] float32 or bfloat16.
+extern "C" int lp_retention_step(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, const float* inv_freq, int rd,
+                                 int interleaved, const int* positions, const float* decays, float q_scale, float norm_eps, float* state,
+                                 const int* slots, void* out, int out_dtype, int B, int H, int dk, int dv, float* zero,
+                                 long long zero_count, cudaStream_t stream) {
+    if (B <= 0) return 0;
+    if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > 512 || dv <= 0) LP_REFUSE("retention_step: %d sequences, %d heads of %d x %d", B, H, dk, dv);
+    if (q_off < 0 || k_off < 0 || v_off < 0 || g_off < 0 || q_off + H * dk > ld || k_off + H * dk > ld || v_off + H * dv > ld || g_off + H * dv > ld)
+        LP_REFUSE("retention_step: columns at %d, %d, %d, %d do not fit rows of %d", q_off, k_off, v_off, g_off, ld);
+    if (rd < 0 || rd > dk || (rd & 1) || (rd > 0 && !inv_freq)) LP_REFUSE("retention_step: a rotation over %d of %d channels", rd, dk);
+    if (((uintptr_t)state & 15) != 0) LP_REFUSE("retention_step: the state must be aligned to 16 bytes");
+    const RetentionArgs a{proj, ld, q_off, k_off, v_off, g_off, inv_freq, rd, interleaved, positions, decays, q_scale, norm_eps, state, slots,
+                          H, dk, dv, zero, zero_count};
+    const size_t smem = ((size_t)2 * dk + 2 * dv) * sizeof(float);
+    if (smem > 46 * 1024) LP_REFUSE("retention_step: heads of %d x %d do not fit shared memory", dk, dv);
+    const dim3 grid(H, B);
+#define LP_RSTEP(KPT, JT)                                                                                                      \
+    do {                                                                                                                       \
+        if (out_dtype == LP_BF16) lp_launch(retention_step_kernel<KPT, JT, __nv_bfloat16>, grid, THREADS, smem, stream, a, (__nv_bfloat16*)out); \
+        else if (out_dtype == LP_F32) lp_launch(retention_step_kernel<KPT, JT, float>, grid, THREADS, smem, stream, a, (float*)out); \
+        else LP_REFUSE("retention_step: output dtype code %d", out_dtype);                                                     \
+    } while (0)
+    if (dk <= 64) LP_RSTEP(4, 4);
+    else if (dk <= 128) LP_RSTEP(8, 4);
+    else if (dk <= 256) LP_RSTEP(16, 2);
+    else LP_RSTEP(32, 1);
+#undef LP_RSTEP
+    return lp_check_launch("retention_step");
+}
+
+// One new token for each of B sequences through a delta rule. proj: float32 [B, ld] (see StepArgs for the columns); out: [B, H * dv] float32 or
 // bfloat16. a_up / g_up null: one decay per head, gate pre-activations straight from the projection.
 extern "C" int lp_delta_step(const float* proj, int ld, int c_off, int b_off, int a_off, int g_off, const float* taps, float* tail,
                              int K, float unit_eps, float q_scale, const float* dt_bias, const float* a_log, const void* a_up,

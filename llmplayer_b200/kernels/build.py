@@ -38,7 +38,7 @@ LIBRARIES: Dict[str, str] = {
     "linear_attention": "linear_attention.cu",
     "routing": "routing.cu",
     "chunked_recurrence": "chunked_recurrence.cu",
-    "delta_step": "delta_step.cu",
+    "recurrent_step": "recurrent_step.cu",
 }
 HEADERS = ("common.cuh", "attention_noalloc.h", "tcgen05_utils.cuh", "attention_decode.cuh")
 

@@ -106,7 +106,9 @@ _SIGNATURES = {
         "lp_chunked_recurrence": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
                                   _P, _P, _P],
     },
-    "delta_step": {
+    "recurrent_step": {
+        "lp_retention_step": [_P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _F, _F, _P, _P, _P, _I, _I, _I, _I, _I, _P,
+                              ctypes.c_longlong, _P],
         "lp_delta_step": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _F, _F, _P, _P, _P, _I, _P, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I,
                           _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
     },
@@ -1620,7 +1622,7 @@ def delta_step(proj: torch.Tensor, columns, taps: torch.Tensor, tail: torch.Tens
                a_up: Optional[torch.Tensor] = None, g_up: Optional[torch.Tensor] = None, gate_sigmoid: bool = False,
                clear: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One token for each sequence through a delta-rule layer, from the projection of its input to the input of its output
-    product, in one kernel (csrc/delta_step.cu): what :func:`short_conv`, :func:`head_unit_norm`, :func:`decay_gates` or
+    product, in one kernel (csrc/recurrent_step.cu): what :func:`short_conv`, :func:`head_unit_norm`, :func:`decay_gates` or
     :func:`low_rank_gates`, :func:`gla_scan` and :func:`gla_finish` do for a step of several tokens. ``proj``: float32 [B, F];
     ``columns`` = (first convolution channel [q | k | v], write strengths, decays, gate); ``out``: [B, H * dv]. ``a_up``
     [H * dk, rank] / ``g_up`` [H * dv, rank]: the decays' / the gate's low-rank maps (``dt_bias`` is then [H * dk])."""
@@ -1649,12 +1651,37 @@ def delta_step(proj: torch.Tensor, columns, taps: torch.Tensor, tail: torch.Tens
     if a_up is not None and g_up is not None and a_up.dtype != g_up.dtype:
         raise KernelError("delta_step: both low-rank maps have one number format")
     c_off, b_off, a_off, g_off = (int(c) for c in columns)
-    lib = library("delta_step")
+    lib = library("recurrent_step")
     _check(lib, lib.lp_delta_step(
         proj.data_ptr(), proj.shape[1], c_off, b_off, a_off, g_off, taps.data_ptr(), tail.data_ptr(), K, float(unit_eps), float(q_scale),
         dt_bias.data_ptr(), a_log.data_ptr(), _ptr(a_up), ranks[0], _ptr(g_up), ranks[1], code, 1 if gate_sigmoid else 0, gain.data_ptr(),
         float(norm_eps), state.data_ptr(), slots.data_ptr(), out.data_ptr(), _code(out, "delta_step out"), B, H, G, dk, dv,
         *_clear_args(clear, "delta_step"), _stream()))
+    return out
+
+
+def retention_step(proj: torch.Tensor, columns, rotation: Rotation, positions: torch.Tensor, decays: torch.Tensor, state: torch.Tensor,
+                   slots: torch.Tensor, norm_eps: float, out: torch.Tensor, *, num_heads: int, key_dim: int, value_dim: int,
+                   q_scale: float, clear: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One token for each sequence through a retention, from the projection of its input to the input of its output product,
+    in one kernel (csrc/recurrent_step.cu): what :func:`gla_scan` (``decay_fixed``, rotated) and :func:`gla_finish` do for a
+    step of several tokens. ``proj``: float32 [B, F]; ``columns`` = (queries, keys, values, gate); ``out``: [B, H * dv]."""
+    _want(proj, "retention_step proj", torch.float32, 2)
+    _want(positions, "retention_step positions", torch.int32, 1)
+    _want(decays, "retention_step decays", torch.float32, 1)
+    _want(state, "retention_step state", torch.float32, 4)
+    _want(slots, "retention_step slots", torch.int32, 1)
+    _want(out, "retention_step out", ndim=2)
+    B, H, dk, dv = slots.numel(), num_heads, key_dim, value_dim
+    if (proj.shape[0] != B or positions.numel() != B or decays.numel() != H or state.shape[1:] != (H, dv, dk) or out.shape != (B, H * dv)):
+        raise KernelError(f"retention_step: proj {tuple(proj.shape)}, state {tuple(state.shape)}, out {tuple(out.shape)}, {B} sequences, "
+                          f"{H} heads of {dk} x {dv}")
+    freq_ptr, rd, interleaved = rotation.checked("retention_step")
+    lib = library("recurrent_step")
+    _check(lib, lib.lp_retention_step(
+        proj.data_ptr(), proj.shape[1], *(int(c) for c in columns), freq_ptr, rd, interleaved, positions.data_ptr(), decays.data_ptr(),
+        float(q_scale), float(norm_eps), state.data_ptr(), slots.data_ptr(), out.data_ptr(), _code(out, "retention_step out"), B, H, dk,
+        dv, *_clear_args(clear, "retention_step"), _stream()))
     return out
 
 

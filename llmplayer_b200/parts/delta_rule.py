@@ -13,10 +13,12 @@ may be the sigmoid of another low-rank map instead of silu(W_g x_t). Each head's
 shared by the heads and by silu(W_g x_t), and projected. State, decays, strengths, unit norms and every sum are float32.
 The recurrence is one more form of the framework's linear-attention scan (csrc/linear_attention.cu): a value column's
 state entries live in the registers of a few threads, and the two read-outs S^T k and S^T q of a token are taken from
-the state before it in one pass of shuffles; prompts of 256 tokens or more run in chunks of 128 side by side (a
-chunk's effect on the state that enters it is S -> P S + L; the first pass forms P, a [key_dim, key_dim] matrix, beside
-L, the chunks' start states follow in order, the second pass writes the outputs). What a sequence carries from step to step is S and the convolutions'
-last taps - 1 inputs. All kernels read the step from device tensors.
+the state before it in one pass of shuffles. Prompts of bfloat16 models run in chunks of 32 tokens whose sums are
+tensor-core products at float32 precision (csrc/chunked_recurrence.cu); steps of one token per sequence run from the
+projection to the gated heads in one kernel (csrc/recurrent_step.cu). float32 prompts of 256 tokens or more run in chunks
+side by side (a chunk's effect on the state that enters it is S -> P S + L; the first pass forms P, a [key_dim, key_dim]
+matrix, beside L, the chunks' start states follow in order, the second pass writes the outputs). What a sequence carries
+from step to step is S and the convolutions' last taps - 1 inputs. All kernels read the step from device tensors.
 """
 from __future__ import annotations
 

@@ -7,7 +7,7 @@ Each head's o_t is RMS-normed over its values with one gain shared by the heads,
 silu(gate x_t), and the heads are projected by ``o``. The state (kept as [heads, value_dim, key_dim]) starts at zero
 (the cache zeroes a slot's row when it is taken) and is carried from step to step; the kernels read the
 row of each sequence's slot from the device, so one-token steps replay from captured graphs
-(csrc/linear_attention.cu).
+(csrc/linear_attention.cu; prompts of bfloat16 models as products over chunks, csrc/chunked_recurrence.cu).
 """
 from __future__ import annotations
 

@@ -7,7 +7,7 @@ square (no gain), the heads are multiplied by silu(W_g x_t) and projected. The r
 framework's linear-attention scan (csrc/linear_attention.cu): one constant decay per head, queries and keys rotated as
 the scan reads them from the projection (the cosines and sines of a step's tokens are formed once and shared by its
 layers), long prompts in chunks side by side. The constant key_dim^-1/2 is applied to the queries, which gives the same
-outputs. What a sequence carries from step to step is S. All kernels read the step from device tensors.
+outputs; one-token steps run from the projection to the gated heads in one kernel (csrc/recurrent_step.cu). What a sequence carries from step to step is S. All kernels read the step from device tensors.
 """
 from __future__ import annotations
 
@@ -104,17 +104,18 @@ class Retention(Part):
         H, dk, dv = s.num_heads, s.key_dim, s.value_dim
         v_off = offset + 2 * self.keys
         g_off = v_off + self.values
-        raw = ctx.buffer("recurrence_raw", (T, self.values), torch.float32)
-        with ops.section("recurrence.scan"):
-            ops.gla_scan(proj, offset, offset + self.keys, v_off, self.decays, cache.rows, ctx.slots, ctx.q_start, raw,
-                         num_heads=H, key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, max_new=ctx.max_new,
-                         scratch=ctx.buffer, decay_fixed=True, rotation=rotation,
-                         angles=ctx.angles(rotation) if rotation.rotary_dim else None, tensor_cores=rt.fast)
         o = ctx.buffer("attn_out", (T, self.values), rt.act_dtype)
-        with ops.section("recurrence.norm"):
-            # an output product that sums partial results wants its target zero: this kernel clears it on the side
-            clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None
-            ops.gla_finish(raw, None, s.norm_eps, proj[:, g_off:g_off + self.values], o, num_heads=H, value_dim=dv, clear=clear)
+        # an output product that sums partial results wants its target zero: the kernel before it clears it on the side
+        clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None
+        if ctx.all_single and dk + dv <= 5800:
+            with ops.section("recurrence.step"):
+                ops.retention_step(proj, (offset, offset + self.keys, v_off, g_off), rotation, ctx.positions, self.decays, cache.rows,
+                                   ctx.slots, s.norm_eps, o, num_heads=H, key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, clear=clear)
+        else:
+            raw = ctx.buffer("recurrence_raw", (T, self.values), torch.float32)
+            self._scan(ctx, cache, proj, (offset, offset + self.keys, v_off), rotation, raw)
+            with ops.section("recurrence.norm"):
+                ops.gla_finish(raw, None, s.norm_eps, proj[:, g_off:g_off + self.values], o, num_heads=H, value_dim=dv, clear=clear)
         if clear is not None:
             ctx.note_cleared()
         with ops.section("recurrence.out"):
@@ -122,6 +123,15 @@ class Retention(Part):
                 self.out.store(o, residual, ctx)
                 return False
             return self.out.accumulate(o, residual, ctx, then_norm)
+
+    def _scan(self, ctx, cache, proj: torch.Tensor, columns, rotation, raw: torch.Tensor) -> None:
+        s, rt = self.spec, self.runtime
+        H, dk, dv = s.num_heads, s.key_dim, s.value_dim
+        with ops.section("recurrence.scan"):
+            ops.gla_scan(proj, *columns, self.decays, cache.rows, ctx.slots, ctx.q_start, raw,
+                         num_heads=H, key_dim=dk, value_dim=dv, q_scale=float(dk) ** -0.5, max_new=ctx.max_new,
+                         scratch=ctx.buffer, decay_fixed=True, rotation=rotation,
+                         angles=ctx.angles(rotation) if rotation.rotary_dim else None, tensor_cores=rt.fast)
 
 
 MIXERS.register("retention", Retention)

@@ -11,7 +11,7 @@ the last one on the token itself, a bias) and silu. Per head h, which reads grou
 y, the heads side by side, is multiplied by silu(z), cut into equal parts that are each divided by their own root mean
 square, multiplied by a gain and projected. The recurrence is the framework's linear-attention scan
 (csrc/linear_attention.cu) with B as keys and C as queries shared by the heads of a group, one decay per head and dt as
-the keys' gain, so long prompts run in chunks side by side like the other recurrences. What a sequence carries from
+the keys' gain; prompts of bfloat16 models run as tensor-core products over chunks (csrc/chunked_recurrence.cu). What a sequence carries from
 step to step is S and the convolution's last taps - 1 inputs. All kernels read the step from device tensors.
 """
 from __future__ import annotations

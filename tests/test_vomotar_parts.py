@@ -354,6 +354,42 @@ def test_single_steps_in_one_kernel(H, G, dk, dv, ra, rg, K, dtype, low_rank):
     assert float((state[1] - 2.0).abs().max()) == 0.0 and float(state[3].abs().max()) == 0.0 and (K == 1 or float((tail[3] - 5.0).abs().max()) == 0.0)
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,dk,dv,rd,decay", [(4, 64, 32, 64, [0.98, 0.995, 0.9985, 0.9995]), (2, 20, 300, 8, [0.5, 1.0]), (1, 128, 256, 128, [0.97]),
+                                              (3, 6, 10, 0, [0.0, 0.9, 0.3]), (2, 256, 24, 2, [0.99, 0.4]), (1, 301, 12, 300, [0.9])])
+def test_single_retention_steps_in_one_kernel(H, dk, dv, rd, decay, dtype):
+    """60 steps of one token for three sequences in slots 4, 0 and 2 that started at positions of their own."""
+    from llmplayer_b200.kernels import ops
+    torch.manual_seed(dk + rd)
+    n, B, off, base = 60, 3, 2, 5000.0
+    freqs = torch.tensor([base ** (-2.0 * i / rd) for i in range(rd // 2)], dtype=torch.float64).float().cuda() if rd else None
+    rotation = ops.Rotation(freqs, rd, False) if rd else ops.NO_ROTATION
+    cols = (off, off + H * dk, off + 2 * H * dk, off + 2 * H * dk + H * dv)
+    x = torch.randn(B, n, cols[3] + H * dv + 3)
+    starts = [0, 7, 100]
+    state = torch.zeros(5, H, dv, dk, device="cuda")
+    state[1] = 2.0
+    junk = torch.full((5000,), 3.0, device="cuda")
+    got = []
+    for t in range(n):
+        out = torch.full((B, H * dv), float("nan"), device="cuda", dtype=dtype)
+        ops.retention_step(x[:, t].contiguous().cuda(), cols, rotation, i32([s + t for s in starts]), torch.tensor(decay).cuda(), state,
+                           i32([4, 0, 2]), 1e-5, out, num_heads=H, key_dim=dk, value_dim=dv, q_scale=dk ** -0.5, clear=junk)
+        got.append(out.float().cpu())
+    got = torch.stack(got, dim=1)
+    assert float(junk.abs().max()) == 0.0 and torch.isfinite(got).all()
+    for b in range(B):
+        p, pos = x[b].double(), torch.arange(n) + starts[b]
+        q = P.rotate_half(p[:, cols[0]:cols[1]].reshape(n, H, dk), pos, base, rd)
+        k = P.rotate_half(p[:, cols[1]:cols[2]].reshape(n, H, dk), pos, base, rd) * dk ** -0.5
+        o, S = P.retention_recurrence(q, k, p[:, cols[2]:cols[3]].reshape(n, H, dv), torch.tensor(decay, dtype=torch.float64))
+        ref = P.unit_rms(o, 1e-5).reshape(n, H * dv) * P.silu(p[:, cols[3]:cols[3] + H * dv])
+        err = float((got[b].double() - ref).abs().max() / ref.abs().max())
+        check_error(f"single retention steps, {dtype}", f"{H} x {dk} x {dv}, rotation {rd}, sequence {b}", err, 1e-4 if dtype == torch.float32 else 5e-3)
+        assert rel(state[[4, 0, 2][b]].transpose(1, 2) * dk ** -0.5, S) < 2e-5
+    assert float((state[1] - 2.0).abs().max()) == 0.0 and float(state[3].abs().max()) == 0.0
+
+
 # --------------------------------------------------------------------------- output gate without a gain
 def test_heads_normed_without_a_gain():
     from llmplayer_b200.kernels import ops
