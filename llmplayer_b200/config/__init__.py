@@ -9,8 +9,9 @@ from .botuvik import BotuvikConfig
 from .zasitar import ZasitarConfig
 from .dopuvik import DopuvikConfig
 from .vomotar import VomotarConfig
+from .zotolix import ZotolixConfig
 
 __all__ = [
-    "ArchitectureConfig", "BotuvikConfig", "DopuvikConfig", "LlamaConfig", "RamupelConfig", "VomotarConfig", "ZasitarConfig", "config_class_for", "config_from_dict",
-    "known_architectures", "load_config", "register_architecture", "unregister_architecture",
+    "ArchitectureConfig", "BotuvikConfig", "DopuvikConfig", "LlamaConfig", "RamupelConfig", "VomotarConfig", "ZasitarConfig", "ZotolixConfig",
+    "config_class_for", "config_from_dict", "known_architectures", "load_config", "register_architecture", "unregister_architecture",
 ]

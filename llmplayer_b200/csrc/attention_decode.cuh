@@ -153,7 +153,14 @@ struct ScoreExtras {
     // dist_scale[h] * ln(1 + dist_rate[h] * n).
     const float* dist_scale;
     const float* dist_rate;
+    // A gate per query token and head: the finished output of head h of token t is multiplied by
+    // sigmoid(gate[t * gate_ld + h]) before it is rounded (null: no gate).
+    const float* gate;
+    int gate_ld;
 };
+__device__ __forceinline__ float head_gate(const ScoreExtras& x, long long token, int head) {
+    return x.gate ? 1.0f / (1.0f + __expf(-__ldcg(x.gate + token * x.gate_ld + head))) : 1.0f;
+}
 // the first position that a query at `pos` sees: by the window, by its chunk (the later of the two)
 __device__ __forceinline__ int first_seen(int pos, int window, const ScoreExtras& x) {
     int lo = window > 0 ? max(0, pos - window + 1) : 0;
@@ -635,7 +642,7 @@ __device__ __forceinline__ void attention_decode_unit(
         }
         if ((FUSED ? shares : num_splits) == 1) {   // the only share: this is the result
             if (l > 0.f) l += sink_term(fused.score, head0 + r, m);
-            out[((size_t)b * H + head0 + r) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+            out[((size_t)b * H + head0 + r) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l * head_gate(fused.score, b, head0 + r) : 0.f);
         } else {
             const size_t slot = ((size_t)b * H + head0 + r) * num_splits + split;
             part_o[slot * hd + d] = acc;
@@ -688,7 +695,7 @@ __device__ __forceinline__ void attention_decode_unit(
                     }
                 }
                 if (l > 0.f) l += sink_term(fused.score, head0 + r, m);
-                out[((size_t)b * H + head0 + r) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+                out[((size_t)b * H + head0 + r) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l * head_gate(fused.score, b, head0 + r) : 0.f);
             }
         }
     }

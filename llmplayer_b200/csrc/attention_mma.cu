@@ -167,7 +167,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
     l_lo += sink_term(extras, h, m_lo); l_hi += sink_term(extras, h, m_hi);
-    const float inv_lo = 1.0f / l_lo, inv_hi = 1.0f / l_hi;
+    const float inv_lo = head_gate(extras, t_begin + row0 + min(r_lo, rows - 1), h) / l_lo;
+    const float inv_hi = head_gate(extras, t_begin + row0 + min(r_hi, rows - 1), h) / l_hi;
 #pragma unroll
     for (int dt = 0; dt < KSTEPS * 2; ++dt) {
         const int d = dt * 8 + (lane & 3) * 2;
@@ -377,7 +378,8 @@ attention_prefill_exact_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat1
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
     l_lo += sink_term(extras, h, m_lo); l_hi += sink_term(extras, h, m_hi);
-    const float inv_lo = 1.0f / l_lo, inv_hi = 1.0f / l_hi;
+    const float inv_lo = head_gate(extras, t_begin + row0 + min(r_lo, rows - 1), h) / l_lo;
+    const float inv_hi = head_gate(extras, t_begin + row0 + min(r_hi, rows - 1), h) / l_hi;
 #pragma unroll
     for (int dt = 0; dt < KSTEPS * 2; ++dt) {
         const int d = dt * 8 + (lane & 3) * 2;
@@ -454,7 +456,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
         }
     }
     if (l > 0.f) l += sink_term(extras, h, m);
-    if (d < hd) out[((size_t)b * H + h) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+    if (d < hd) out[((size_t)b * H + h) * hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l * head_gate(extras, b, h) : 0.f);
 }
 
 // Opt in to `bytes` of dynamic shared memory; remembered per kernel so that later calls
@@ -493,10 +495,14 @@ int check_geometry(const char* what, int H, int G, int hd) {
 }
 
 // softcap > 0: scores are capped at it; sinks: float32 [H] or null (see ScoreExtras)
-// chunk > 0: keys of the query's own chunk only; dist_scale, dist_rate: float32 [H] each, or both null
+// chunk > 0: keys of the query's own chunk only; dist_scale, dist_rate: float32 [H] each, or both null; gate: float32, a
+// row of gate_ld values per query token whose first H are the heads' gates, or null
 static ScoreExtras make_extras(float scale, float softcap, const float* sinks, int keep = 0, int chunk = 0,
-                               const float* dist_scale = nullptr, const float* dist_rate = nullptr) {
+                               const float* dist_scale = nullptr, const float* dist_rate = nullptr, const float* gate = nullptr,
+                               int gate_ld = 0) {
     ScoreExtras x{};
+    x.gate = gate;
+    x.gate_ld = gate_ld;
     x.chunk = chunk > 0 ? chunk : 0;
     x.dist_scale = dist_scale;
     x.dist_rate = dist_rate;
@@ -517,9 +523,10 @@ extern "C" int lp_attention_prefill(const void* q, void* out, const void* pages,
                                     const int* q_start, const int* kv_len, int B, int max_new, int H, int G, int hd,
                                     int page_size, float scale, int window, float softcap, const float* sinks,
                                     int split_weights, int keep, int chunk, const float* dist_scale,
-                                    const float* dist_rate, cudaStream_t stream) {
+                                    const float* dist_rate, const float* gate, int gate_ld, cudaStream_t stream) {
     if (B <= 0 || max_new <= 0) return 0;
-    const ScoreExtras extras = make_extras(scale, softcap, sinks, keep, chunk, dist_scale, dist_rate);
+    if (gate && gate_ld < H) LP_REFUSE("attention_prefill: rows of %d gates for %d heads", gate_ld, H);
+    const ScoreExtras extras = make_extras(scale, softcap, sinks, keep, chunk, dist_scale, dist_rate, gate, gate_ld);
     int rc = check_geometry("attention_prefill", H, G, hd);
     if (rc) return rc;
     rc = check_shaping("attention_prefill", window > 0 ? keep : 0, chunk, dist_scale, dist_rate, split_weights);
@@ -606,11 +613,13 @@ static int attention_decode_launch(const void* q, void* out, const void* pages, 
                                    const int* kv_len, float* scratch, int B, int H, int G, int hd, int page_size,
                                    float scale, int window, int pages_per_split, int num_splits, int min_share_pages,
                                    float softcap, const float* sinks, int split_weights, cudaStream_t stream, int keep = 0,
-                                   int chunk = 0, const float* dist_scale = nullptr, const float* dist_rate = nullptr) {
+                                   int chunk = 0, const float* dist_scale = nullptr, const float* dist_rate = nullptr,
+                                   const float* gate = nullptr, int gate_ld = 0) {
     if (B <= 0) return 0;
+    if (gate && gate_ld < H) LP_REFUSE("attention_decode: rows of %d gates for %d heads", gate_ld, H);
     if (keep > 0 && min_share_pages <= 0) LP_REFUSE("attention_decode: kept first tokens need shares fitted to the sequence (%d)", keep);
     FusedDecodeArgs plain_args{};
-    plain_args.score = make_extras(scale, softcap, sinks, window > 0 ? keep : 0, chunk, dist_scale, dist_rate);
+    plain_args.score = make_extras(scale, softcap, sinks, window > 0 ? keep : 0, chunk, dist_scale, dist_rate, gate, gate_ld);
     int rc = check_geometry("attention_decode", H, G, hd);
     if (rc) return rc;
     rc = check_shaping("attention_decode", window > 0 ? keep : 0, chunk, dist_scale, dist_rate, split_weights);
@@ -671,11 +680,12 @@ extern "C" int lp_attention_decode_fitted(const void* q, void* out, const void* 
                                           int pt_stride, const int* kv_len, float* scratch, int B, int H, int G, int hd,
                                           int page_size, float scale, int window, int num_splits, int min_share_pages,
                                           float softcap, const float* sinks, int split_weights, int keep, int chunk,
-                                          const float* dist_scale, const float* dist_rate, cudaStream_t stream) {
+                                          const float* dist_scale, const float* dist_rate, const float* gate, int gate_ld,
+                                          cudaStream_t stream) {
     if (min_share_pages <= 0) LP_REFUSE("attention_decode_fitted: shares of at least %d pages", min_share_pages);
     return attention_decode_launch(q, out, pages, page_table, pt_stride, kv_len, scratch, B, H, G, hd, page_size, scale,
                                    window, pt_stride > 0 ? pt_stride : 1, num_splits, min_share_pages, softcap, sinks,
-                                   split_weights, stream, keep, chunk, dist_scale, dist_rate);
+                                   split_weights, stream, keep, chunk, dist_scale, dist_rate, gate, gate_ld);
 }
 
 // Decode attention that starts from the fused projection output: rotation of queries and of the new key,

@@ -23,7 +23,8 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
                        const int* __restrict__ page_table, int pt_stride, const int* __restrict__ seq_ids,
                        const int* __restrict__ positions, int H, int G, int hd, int page_size, float scale,
                        int window, float softcap, const float* __restrict__ sinks, int keep, int chunk,
-                       const float* __restrict__ dist_scale, const float* __restrict__ dist_rate) {
+                       const float* __restrict__ dist_scale, const float* __restrict__ dist_rate,
+                       const float* __restrict__ gate, int gate_ld) {
     __shared__ float qs[MAX_HD];
     __shared__ float prob[KB];
     __shared__ long long row_off[KB];
@@ -97,7 +98,8 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
         acc0 *= alpha;
         acc1 *= alpha;
     }
-    const float inv = 1.0f / l;
+    // a gate per query token and head multiplies the head's finished output
+    const float inv = gate ? 1.0f / (l * (1.0f + expf(-gate[(long long)t * gate_ld + h]))) : 1.0f / l;
     TQ* o = out + ((long long)t * H + h) * hd;
     if (tid < hd) o[tid] = lp_from_float<TQ>(acc0 * inv);
     if (tid + KB < hd) o[tid + KB] = lp_from_float<TQ>(acc1 * inv);
@@ -110,13 +112,15 @@ attention_plain_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TKV
 // softcap * tanh(s / softcap) after the scale. sinks (optional): float32 [H], see the kernel. keep > 0 (with a window):
 // the sequence's first `keep` tokens stay visible to every later query, at their true positions. chunk > 0: a query at p
 // sees keys from p / chunk * chunk on only. dist_scale, dist_rate (optional, float32 [H] each): a key n positions back
-// loses dist_scale[h] * ln(1 + dist_rate[h] * n) of its score.
+// loses dist_scale[h] * ln(1 + dist_rate[h] * n) of its score. gate (optional, float32, rows of gate_ld values): head h's
+// output of query token t is multiplied by sigmoid(gate[t, h]).
 extern "C" int lp_attention_plain(const void* q, void* out, int q_dtype, const void* pages, int kv_dtype,
                                   const int* page_table, int pt_stride, const int* seq_ids, const int* positions,
                                   int T, int H, int G, int hd, int page_size, float scale, int window,
                                   float softcap, const float* sinks, int keep, int chunk, const float* dist_scale,
-                                  const float* dist_rate, cudaStream_t stream) {
+                                  const float* dist_rate, const float* gate, int gate_ld, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (gate && gate_ld < H) LP_REFUSE("attention_plain: rows of %d gates for %d heads", gate_ld, H);
     if ((dist_scale == nullptr) != (dist_rate == nullptr)) LP_REFUSE("attention_plain: a distance bias has a scale and a rate per head");
     if (keep > 0 && window > 0 && chunk > 0) LP_REFUSE("attention_plain: kept first tokens (%d) and chunks (%d) exclude each other", keep, chunk);
     if (H <= 0 || G <= 0 || H % G) LP_REFUSE("attention_plain: %d query heads over %d key heads", H, G);
@@ -128,7 +132,7 @@ extern "C" int lp_attention_plain(const void* q, void* out, int q_dtype, const v
     attention_plain_kernel<TQ, TKV><<<grid, KB, 0, stream>>>((const TQ*)q, (TQ*)out, (const TKV*)pages,          \
                                                              page_table, pt_stride, seq_ids, positions, H, G,  \
                                                              hd, page_size, scale, window, softcap, sinks, keep, \
-                                                             chunk, dist_scale, dist_rate)
+                                                             chunk, dist_scale, dist_rate, gate, gate_ld)
     if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_LAUNCH_ATT(float, float);
     else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_LAUNCH_ATT(__nv_bfloat16, __nv_bfloat16);
     else if (q_dtype == LP_F32 && kv_dtype == LP_BF16) LP_LAUNCH_ATT(float, __nv_bfloat16);

@@ -644,7 +644,9 @@ extern "C" int lp_advance(int* tokens, int* positions, int* kv_len, const int* s
 // sequence that holds its position, pages[page][0|1][g][position % page_size][:hdp]. A warp per head; all float32.
 // `qgain` / `kgain` (optional, [dk], shared by the heads): BEFORE the rotation every query / key head is RMS-normed
 // over dk with that gain and `gain_eps` inside the root. `vnorm`: every value head is divided by its root mean square over
-// dv (`vnorm_eps` inside the root). G = 0 with `pages` null: a layer that has queries only.
+// dv (`vnorm_eps` inside the root). G = 0 with `pages` null: a layer that has queries only. `vkeep` (optional, float32
+// [T, G * dv]): the values of this layer, with their bias, are left there for later layers of the step. `vfirst` (the same
+// buffer, in a later layer) with `vmix` (one number lambda): a value becomes (1 - lambda) v + lambda vfirst before it is stored.
 constexpr int PREP_MAX = 256;
 template <typename TQ, typename TKV>
 __global__ void __launch_bounds__(256)
@@ -653,7 +655,8 @@ qkv_prepare_kernel(const float* __restrict__ qkv, int ld, const float* __restric
                    int pt_stride, TQ* __restrict__ q_out, TKV* __restrict__ pages, int H, int G, int dk, int dv, int hdp,
                    int rd, int interleaved, int unit, float unit_eps, int page_size, float* __restrict__ zero,
                    long long zero_count, const float* __restrict__ qgain, const float* __restrict__ kgain, float gain_eps,
-                   int vnorm, float vnorm_eps) {
+                   int vnorm, float vnorm_eps, float* __restrict__ vkeep, const float* __restrict__ vfirst,
+                   const float* __restrict__ vmix) {
     __shared__ float cs[PREP_MAX];
     __shared__ float buf[8][PREP_MAX];
     lp_grid_release();
@@ -726,8 +729,17 @@ qkv_prepare_kernel(const float* __restrict__ qkv, int ld, const float* __restric
                 }
                 factor = 1.0f / sqrtf(lp_warp_sum(ss) / (float)dv + vnorm_eps);
             }
-            for (int e = lane; e < hdp; e += 32)
-                dst[e] = lp_from_float<TKV>(e < dv ? (row[src + e] + (bias ? bias[src + e] : 0.f)) * factor : 0.f);
+            const float lambda = vfirst ? *vmix : 0.f;
+            const long long at = ((long long)t * G + g) * dv;            // this value head in the buffer of a step's first values
+            for (int e = lane; e < hdp; e += 32) {
+                float val = 0.f;
+                if (e < dv) {
+                    val = (row[src + e] + (bias ? bias[src + e] : 0.f)) * factor;
+                    if (vkeep) vkeep[at + e] = val;
+                    if (vfirst) val = (1.0f - lambda) * val + lambda * vfirst[at + e];
+                }
+                dst[e] = lp_from_float<TKV>(val);
+            }
         }
     }
 }
@@ -737,8 +749,9 @@ extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const
                               void* pages, int kv_dtype, int T, int H, int G, int dk, int dv, int hdp, int rd,
                               int interleaved, int unit, float unit_eps, int page_size, float* zero, long long zero_count,
                               const float* qgain, const float* kgain, float gain_eps, int vnorm, float vnorm_eps,
-                              cudaStream_t stream) {
+                              float* vkeep, const float* vfirst, const float* vmix, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (vfirst && !vmix) LP_REFUSE("qkv_prepare: first values without the share they get");
     if (H <= 0 || G < 0 || dk <= 0 || dv <= 0) LP_REFUSE("qkv_prepare: %d / %d heads of %d and %d", H, G, dk, dv);
     if (hdp < dk || hdp < dv || dk > PREP_MAX) LP_REFUSE("qkv_prepare: heads of %d and %d stored in %d (at most %d)", dk, dv, hdp, PREP_MAX);
     if (rd < 0 || rd > dk || (rd & 1)) LP_REFUSE("qkv_prepare: rotary width %d for heads of %d", rd, dk);
@@ -749,7 +762,7 @@ extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const
 #define LP_LAUNCH_PREP(TQ, TKV)                                                                                       \
     lp_launch(qkv_prepare_kernel<TQ, TKV>, T, 256, 0, stream, qkv, ld, bias, inv_freq, positions, seq_ids, page_table, \
               pt_stride, (TQ*)q_out, (TKV*)pages, H, G, dk, dv, hdp, rd, interleaved, unit, unit_eps, page_size, zero,  \
-              zero_count, qgain, kgain, gain_eps, vnorm, vnorm_eps)
+              zero_count, qgain, kgain, gain_eps, vnorm, vnorm_eps, vkeep, vfirst, vmix)
     if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_LAUNCH_PREP(float, float);
     else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_LAUNCH_PREP(__nv_bfloat16, __nv_bfloat16);
     else LP_REFUSE("qkv_prepare: dtype codes q=%d kv=%d", q_dtype, kv_dtype);

@@ -137,23 +137,14 @@ expert_scale_vec8_kernel(__nv_bfloat16* __restrict__ hidden, int ldh, const floa
 
 
 // Another rule: the `top` experts with the largest logits z[e] + bias[e] are chosen, and their weights are the softmax
-// over the chosen logits alone. A warp per token; among equal logits the expert with the lower index wins. `extra`
-// further columns of z (beyond the E logits) are gates of experts that every token uses: weights[t, E + i] =
-// sigmoid(z[t, E + i]).
-__global__ void __launch_bounds__(128)
-route_top_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, float* __restrict__ weights, int ldw,
-                 int T, int E, int top, int extra) {
-    extern __shared__ float sm[];
-    lp_grid_release();
-    lp_grid_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const long long t = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
-    if (t >= T) return;
-    float* s = sm + (size_t)warp * 2 * E;
-    float* w = s + E;
+// over the chosen logits alone (form 0) or the sigmoid of each chosen logit (form 1, not renormalised). One warp per token;
+// among equal logits the expert with the lower index wins. s, w: E floats of shared memory each; w holds the weights
+// afterwards (zero for experts that were not chosen). Called by a whole warp.
+__device__ __forceinline__ void choose_top(const float* __restrict__ z, const float* __restrict__ bias, float* s, float* w, int E,
+                                           int top, int form, int lane) {
     for (int e = lane; e < E; e += 32) {
-        s[e] = z[t * ldz + e] + (bias ? bias[e] : 0.f);
-        w[e] = 0.f;
+        s[e] = z[e] + (bias ? bias[e] : 0.f);
+        w[e] = -1.f;                                        // not chosen (weights are never negative)
     }
     __syncwarp();
     float big = 0.f, sum = 0.f;
@@ -162,7 +153,7 @@ route_top_kernel(const float* __restrict__ z, int ldz, const float* __restrict__
         float bv = -INFINITY;
         int best = E;
         for (int e = lane; e < E; e += 32)
-            if (w[e] == 0.f && s[e] > bv) { bv = s[e]; best = e; }
+            if (w[e] < 0.f && s[e] > bv) { bv = s[e]; best = e; }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
@@ -171,14 +162,89 @@ route_top_kernel(const float* __restrict__ z, int ldz, const float* __restrict__
         }
         if (best >= E) break;
         if (n == 0) big = bv;
-        const float p = expf(bv - big);
+        const float p = form == 0 ? expf(bv - big) : 1.0f / (1.0f + expf(-bv));
         sum += p;
         if (lane == 0) w[best] = p;
         __syncwarp();
     }
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < E; e += 32) weights[t * ldw + e] = w[e] * inv;
+    const float inv = form == 0 ? 1.0f / sum : 1.0f;
+    for (int e = lane; e < E; e += 32) w[e] = w[e] < 0.f ? 0.f : w[e] * inv;
+    __syncwarp();
+}
+
+// A warp per token. `extra` further columns of z (beyond the E logits) are gates of experts that every token uses:
+// weights[t, E + i] = sigmoid(z[t, E + i]).
+__global__ void __launch_bounds__(128)
+route_top_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, float* __restrict__ weights, int ldw,
+                 int T, int E, int top, int extra, int form) {
+    extern __shared__ float sm[];
+    lp_grid_release();
+    lp_grid_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const long long t = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= T) return;
+    float* s = sm + (size_t)warp * 2 * E;
+    float* w = s + E;
+    choose_top(z + t * ldz, bias, s, w, E, top, form, lane);
+    for (int e = lane; e < E; e += 32) weights[t * ldw + e] = w[e];
     for (int i = lane; i < extra; i += 32) weights[t * ldw + E + i] = 1.0f / (1.0f + expf(-z[t * ldz + E + i]));
+}
+
+// Hidden activations of ungated squared-ReLU experts from the float32 sums of ONE stacked up product over all experts:
+// z[t, c] with c / ff the expert. on_input: a token's weight w multiplies the expert's input, so that
+// hidden = max(w z, 0)^2; else its output: hidden = w max(z, 0)^2. The weights come from `weights` [T, ldw], or (`top` > 0)
+// are formed here from the token's E router logits, which are columns E * ff .. of the same product: every block chooses
+// for its own token (choose_top without a bias), so that no kernel stands between the product and its activation.
+// A token per blockIdx.y (and every gridDim.y-th one after it); VEC: four columns per thread (rows on 16-byte boundaries,
+// expert sizes of a multiple of four).
+template <typename TH, int VEC>
+__global__ void __launch_bounds__(256)
+expert_relu2_kernel(const float* __restrict__ z, int ldz, TH* __restrict__ hidden, const float* __restrict__ weights, int ldw,
+                    int T, int E, int ff, int on_input, int top, int form, float* __restrict__ zero, long long zero_count) {
+    extern __shared__ float sm[];            // scores [E], weights [E]
+    lp_grid_release();
+    lp_grid_wait();
+    clear_on_the_side(zero, zero_count);
+    float* w = sm + E;
+    const int total = E * ff;
+    for (long long t = blockIdx.y; t < T; t += gridDim.y) {
+        const float* row = z + t * ldz;
+        __syncthreads();
+        if (top > 0) {
+            if (threadIdx.x < 32) choose_top(row + total, nullptr, sm, w, E, top, form, threadIdx.x);
+        } else {
+            for (int e = threadIdx.x; e < E; e += blockDim.x) w[e] = weights[t * ldw + e];
+        }
+        __syncthreads();
+        for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < total / VEC; i += gridDim.x * blockDim.x) {
+            const int c = i * VEC;
+            const float we = w[c / ff];
+            const float in = on_input ? we : 1.0f, after = on_input ? 1.0f : we;
+            if constexpr (VEC == 4) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (we != 0.f) {                         // an expert that was not chosen: its sums are not even read
+                    const float4 z4 = *reinterpret_cast<const float4*>(row + c);
+                    v[0] = z4.x; v[1] = z4.y; v[2] = z4.z; v[3] = z4.w;
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const float r = fmaxf(in * v[k], 0.f);
+                        v[k] = r * r * after;
+                    }
+                }
+                if constexpr (sizeof(TH) == 2) {
+                    uint2 packed;
+                    *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v[0], v[1]);
+                    *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v[2], v[3]);
+                    *reinterpret_cast<uint2*>(hidden + t * total + c) = packed;
+                } else {
+                    *reinterpret_cast<float4*>(hidden + t * total + c) = make_float4(v[0], v[1], v[2], v[3]);
+                }
+            } else {
+                const float r = we != 0.f ? fmaxf(in * row[c], 0.f) : 0.f;
+                hidden[t * total + c] = lp_from_float<TH>(r * r * after);
+            }
+        }
+    }
 }
 
 // Hidden activations of clamped gated experts from the float32 sums of ONE stacked product over all experts:
@@ -379,16 +445,41 @@ extern "C" int lp_expert_scale(void* hidden, int dtype, int ldh, const float* we
 }
 
 // z: float32 [T, ldz] (E logits per row, then `extra` gate columns); bias: float32 [E] or null; weights: float32
-// [T, ldw], E + extra values per row written.
+// [T, ldw], E + extra values per row written. form 0: softmax over the chosen logits; form 1: their sigmoids.
 extern "C" int lp_route_top(const float* z, int ldz, const float* bias, float* weights, int ldw, int T, int E, int top,
-                            int extra, cudaStream_t stream) {
+                            int extra, int form, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (E <= 0 || top <= 0 || top > E || extra < 0) LP_REFUSE("route_top: %d of %d experts, %d gates", top, E, extra);
+    if (form != 0 && form != 1) LP_REFUSE("route_top: form %d", form);
     if (ldz < E + extra || ldw < E + extra) LP_REFUSE("route_top: rows of %d and %d values for %d columns", ldz, ldw, E + extra);
     const size_t smem = (size_t)4 * 2 * E * sizeof(float);
     if (smem > 48 * 1024) LP_REFUSE("route_top: %d experts need %zu bytes of shared memory", E, smem);
-    lp_launch(route_top_kernel, (unsigned)((T + 3) / 4), 128, smem, stream, z, ldz, bias, weights, ldw, T, E, top, extra);
+    lp_launch(route_top_kernel, (unsigned)((T + 3) / 4), 128, smem, stream, z, ldz, bias, weights, ldw, T, E, top, extra, form);
     return lp_check_launch("route_top");
+}
+
+// z: float32 [T, ldz]: E * ff up sums per row, and (top > 0) the E router logits behind them; hidden: [T, E * ff] (dtype
+// code); weights (top == 0): float32 [T, ldw]. zero: a float32 buffer cleared on the side.
+extern "C" int lp_expert_relu2(const float* z, int ldz, void* hidden, int dtype, const float* weights, int ldw, int T, int E,
+                               int ff, int on_input, int top, int form, float* zero, long long zero_count, cudaStream_t stream) {
+    if (T <= 0 || E <= 0 || ff <= 0) return 0;
+    if (top < 0 || top > E || (form != 0 && form != 1)) LP_REFUSE("expert_relu2: %d of %d experts, form %d", top, E, form);
+    if (top == 0 && (!weights || ldw < E)) LP_REFUSE("expert_relu2: rows of %d weights for %d experts", ldw, E);
+    if (ldz < E * ff + (top > 0 ? E : 0)) LP_REFUSE("expert_relu2: rows of %d values for %d experts of %d", ldz, E, ff);
+    if (dtype != LP_F32 && dtype != LP_BF16) LP_REFUSE("expert_relu2: dtype code %d", dtype);
+    const size_t smem = (size_t)2 * E * sizeof(float);
+    if (smem > 48 * 1024) LP_REFUSE("expert_relu2: %d experts need %zu bytes of shared memory", E, smem);
+    const bool vec = ff % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)hidden) & 15) == 0;
+    int bx = (E * ff / (vec ? 4 : 1) + 255) / 256;
+    if (bx > 64) bx = 64;
+    const dim3 grid(bx, T < 65535 ? T : 65535);
+#define LP_EXPERT_RELU2(TH, V)                                                                                           \
+    lp_launch(expert_relu2_kernel<TH, V>, grid, 256, smem, stream, z, ldz, (TH*)hidden, weights, ldw, T, E, ff, on_input, \
+              top, form, zero, zero_count)
+    if (dtype == LP_F32) { if (vec) LP_EXPERT_RELU2(float, 4); else LP_EXPERT_RELU2(float, 1); }
+    else { if (vec) LP_EXPERT_RELU2(__nv_bfloat16, 4); else LP_EXPERT_RELU2(__nv_bfloat16, 1); }
+#undef LP_EXPERT_RELU2
+    return lp_check_launch("expert_relu2");
 }
 
 // z: float32 [T, ldz] with the gate sums of `total` hidden columns, then their up sums; hidden: [T, total].

@@ -32,6 +32,10 @@ class Model:
                 raise ConfigError(f"run {i} names layer {run.layer}, the model has {len(self.blocks)}")
             if run.reads_cache_of is not None and not 0 <= run.reads_cache_of < i:
                 raise ConfigError(f"run {i} reads the cache of run {run.reads_cache_of}, which does not precede it")
+            if i and (run.add_embedding or run.add_vector is not None) and all(
+                    getattr(self.blocks[r.layer], "kind_bundle", False) for r in (self.runs[i - 1], run)):
+                raise ConfigError(f"run {i} adds to the stream between two layers that keep a bundle of streams")
+        self._check_shown_values()
         self.runtime: Optional[Runtime] = None
         # what some runs add to the stream before they start: the embedding's output, a row of a learned table
         self._keeps_embedding = any(run.add_embedding for run in self.runs)
@@ -44,6 +48,17 @@ class Model:
         self._vectors: Dict[str, torch.Tensor] = {}
         # blocks whose forward takes (normed_ready, next_block) can hand a fused norm to the next block
         self._chains = ["next_block" in inspect.signature(b.forward).parameters for b in self.blocks]
+
+    def _check_shown_values(self) -> None:
+        """A layer that blends an earlier layer's values into its own finds them shown by a run before it, in its size."""
+        shown = None
+        for i, run in enumerate(self.runs):
+            spec = getattr(self.layout.layers[run.layer], "mixer", None)
+            size = getattr(spec, "num_kv_heads", 0) * (getattr(spec, "value_dim", None) or getattr(spec, "head_dim", 0))
+            if getattr(spec, "value_blend", None) is not None and shown != size:
+                raise ConfigError(f"run {i} blends {size} values per token, the runs before it show {shown or 'none'}")
+            if getattr(spec, "shows_values", False):
+                shown = size
 
     @property
     def capture_safe(self) -> bool:

@@ -39,6 +39,7 @@ LIBRARIES: Dict[str, str] = {
     "routing": "routing.cu",
     "chunked_recurrence": "chunked_recurrence.cu",
     "recurrent_step": "recurrent_step.cu",
+    "stream_bundle": "stream_bundle.cu",
 }
 HEADERS = ("common.cuh", "attention_noalloc.h", "tcgen05_utils.cuh", "attention_decode.cuh")
 

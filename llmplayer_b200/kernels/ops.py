@@ -33,7 +33,7 @@ _SIGNATURES = {
         "lp_advance": [_P, _P, _P, _P, _I, _P],
         "lp_rope_angles": [_P, _P, _P, _I, _I, _P],
         "lp_qkv_prepare": [_P, _I, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P,
-                           ctypes.c_longlong, _P, _P, _F, _I, _F, _P],
+                           ctypes.c_longlong, _P, _P, _F, _I, _F, _P, _P, _P, _P],
         "lp_pair_norm_add": [_P, _P, _F, _F, _P, _P, _F, _F, _P, _P, _F, _I, _P, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_post_norm_add": [_P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P, ctypes.c_longlong, _P, _P, _P],
         "lp_gated_act": [_P, _I, _P, _P, _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
@@ -44,7 +44,8 @@ _SIGNATURES = {
     "routing": {
         "lp_route": [_P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
         "lp_expert_scale": [_P, _I, _I, _P, _I, _I, _I, _I, _P, ctypes.c_longlong, _P, _P, _I, _I, _I, _I, _P],
-        "lp_route_top": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+        "lp_route_top": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+        "lp_expert_relu2": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_expert_act": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P, ctypes.c_longlong, _P],
         "lp_route_softmax": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P],
         "lp_identity_experts": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P],
@@ -53,7 +54,7 @@ _SIGNATURES = {
         "lp_gemm_plain": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "attention_plain": {
-        "lp_attention_plain": [_P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _P, _P, _P],
+        "lp_attention_plain": [_P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _P, _P, _P, _I, _P],
     },
     "gemm_tcgen05": {
         "lp_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P,
@@ -64,9 +65,9 @@ _SIGNATURES = {
         "lp_gemm_qkv_rope": [_P, _P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P],
     },
     "attention_mma": {
-        "lp_attention_prefill": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _I, _P, _P, _P],
+        "lp_attention_prefill": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P, _I, _I, _I, _P, _P, _P, _I, _P],
         "lp_attention_decode": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _P],
-        "lp_attention_decode_fitted": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P],
+        "lp_attention_decode_fitted": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P, _I, _P],
         "lp_attention_decode_fused": [_P, _I, _P, _I, _I, _P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I,
                                       _I, _I, _I, _P, _F, _I, ctypes.c_longlong, _P, _P],
     },
@@ -111,6 +112,9 @@ _SIGNATURES = {
                               ctypes.c_longlong, _P],
         "lp_delta_step": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _F, _F, _P, _P, _P, _I, _P, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I,
                           _I, _I, _I, _I, _P, ctypes.c_longlong, _P],
+    },
+    "stream_bundle": {
+        "lp_stream_bundle": [_P, _I, _P, _P, _P, _F, _P, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P, ctypes.c_longlong, _P],
     },
     "host_loop": {
         "lp_decode_loop": [_P, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P],
@@ -899,14 +903,16 @@ def gemm_few(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = ST
 def attention_plain(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, page_table: torch.Tensor,
                     seq_ids: torch.Tensor, positions: torch.Tensor, *, num_heads: int, num_kv_heads: int,
                     head_dim: int, scale: float, window: Optional[int], softcap: Optional[float] = None,
-                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, distance=None, gate=None) -> torch.Tensor:
     """Each query token attends over the cached keys of its sequence up to its own
     position (and within ``window``, if given). ``softcap``: scores become softcap * tanh(score / softcap) after the
     scale; ``sinks``: float32 [H], a logit per head that enters the softmax's denominator once. ``keep_first`` (with a
     window): the sequence's first ``keep_first`` tokens stay visible to every later query. ``chunk`` > 0: a query at
     position p sees keys of its own chunk only, from p // chunk * chunk on. ``distance`` = (scale, rate), float32 [H] each:
-    the score of a key n positions back loses scale[h] * ln(1 + rate[h] * n)."""
+    the score of a key n positions back loses scale[h] * ln(1 + rate[h] * n). ``gate``: float32 [T, H] (may be a column
+    slice): head h's output of token t is multiplied by sigmoid(gate[t, h])."""
     dist_scale, dist_rate = _distance_args(distance, num_heads, "attention")
+    gate_ptr, gate_ld = _gate_args(gate, q.shape[0], num_heads, "attention")
     _check_sinks(sinks, num_heads, "attention")
     _want(q, "attention q", ndim=2)
     _want(out, "attention out", q.dtype, 2)
@@ -925,8 +931,18 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pag
         q.data_ptr(), out.data_ptr(), _code(q, "attention q"), pages.data_ptr(), _code(pages, "attention pages"),
         page_table.data_ptr(), page_table.shape[1], seq_ids.data_ptr(), positions.data_ptr(), T, H, G, hd,
         pages.shape[3], float(scale), int(window) if window else 0, float(softcap or 0.0), _ptr(sinks),
-        int(keep_first) if window else 0, int(chunk or 0), dist_scale, dist_rate, _stream()))
+        int(keep_first) if window else 0, int(chunk or 0), dist_scale, dist_rate, gate_ptr, gate_ld, _stream()))
     return out
+
+
+def _gate_args(gate: Optional[torch.Tensor], tokens: int, num_heads: int, what: str):
+    """(pointer, row length) of a gate per token and head, or (None, 0)."""
+    if gate is None:
+        return None, 0
+    ptr, ld = _slice(gate, f"{what} gate")
+    if gate.shape != (tokens, num_heads):
+        raise KernelError(f"{what}: gates {tuple(gate.shape)} for {tokens} tokens and {num_heads} heads")
+    return ptr, ld
 
 
 def _distance_args(distance, num_heads: int, what: str):
@@ -965,14 +981,15 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
                       q_start: torch.Tensor, kv_len: torch.Tensor, max_new: int, *, num_heads: int,
                       num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
                       softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-                      exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
+                      exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None, gate=None) -> torch.Tensor:
     """Tensor-core attention for a step that brings several tokens per sequence. ``keep_first`` (with a window): the
     sequence's first ``keep_first`` tokens stay visible to every later query.
     ``q_start`` [B+1]: offsets of each sequence's new tokens; ``kv_len`` [B]: lengths after the step.
     ``exact_weights``: the softmax weights enter the product with the values at float32 precision (as a bfloat16
     value plus a bfloat16 rest, two products) instead of rounded to bfloat16. ``chunk``, ``distance`` (with
-    ``exact_weights``): see :func:`attention_plain`."""
+    ``exact_weights``), ``gate``: see :func:`attention_plain`."""
     dist_scale, dist_rate = _distance_args(distance, num_heads, "attention_prefill")
+    gate_ptr, gate_ld = _gate_args(gate, q.shape[0], num_heads, "attention_prefill")
     _check_attention(q, out, pages, page_table, num_heads, num_kv_heads, head_dim, "attention_prefill")
     _want(q_start, "attention_prefill q_start", torch.int32, 1)
     _want(kv_len, "attention_prefill kv_len", torch.int32, 1)
@@ -982,7 +999,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
     _check_sinks(sinks, num_heads, "attention_prefill")
     keep_first = int(keep_first) if window else 0
     if (head_dim in (64, 128) and max_new > 64 and tcgen05_attention and not softcap and sinks is None and not exact_weights
-            and not keep_first and not chunk and distance is None):
+            and not keep_first and not chunk and distance is None and gate is None):
         # long runs of new tokens with heads of 64 or 128: scores and P V on the tcgen05 tensor cores
         lib = library("attention_tcgen05")
         _check(lib, lib.lp_attention_prefill_tc(
@@ -996,7 +1013,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, p
         q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1],
         q_start.data_ptr(), kv_len.data_ptr(), B, int(max_new), num_heads, num_kv_heads, head_dim, pages.shape[3],
         float(scale), int(window) if window else 0, float(softcap or 0.0), _ptr(sinks), 1 if exact_weights else 0,
-        keep_first, int(chunk or 0), dist_scale, dist_rate, _stream()))
+        keep_first, int(chunk or 0), dist_scale, dist_rate, gate_ptr, gate_ld, _stream()))
     return out
 
 
@@ -1026,12 +1043,14 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
                      kv_len: torch.Tensor, scratch, *, num_heads: int, num_kv_heads: int, head_dim: int,
                      scale: float, window: Optional[int], pages_per_split: int = 0, num_splits: int = 0,
                      softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-                     exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
+                     exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None, gate=None) -> torch.Tensor:
     """Tensor-core attention for a step of one token per sequence. ``scratch(name, shape, dtype)``
     supplies the float32 buffer for the partial results of the shares. ``keep_first`` (with a window, shares fitted to
     the sequences): the sequence's first ``keep_first`` tokens stay visible; their pages are visited first. ``chunk``,
-    ``distance`` (shares fitted to the sequences, ``exact_weights``): see :func:`attention_plain`."""
+    ``distance`` (shares fitted to the sequences, ``exact_weights``), ``gate`` (shares fitted to the sequences): see
+    :func:`attention_plain`."""
     dist_scale, dist_rate = _distance_args(distance, num_heads, "attention_decode")
+    gate_ptr, gate_ld = _gate_args(gate, q.shape[0], num_heads, "attention_decode")
     _check_attention(q, out, pages, page_table, num_heads, num_kv_heads, head_dim, "attention_decode")
     _want(kv_len, "attention_decode kv_len", torch.int32, 1)
     _check_sinks(sinks, num_heads, "attention_decode")
@@ -1040,8 +1059,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
         raise KernelError(f"attention_decode: {B} sequences, q {tuple(q.shape)}, table {tuple(page_table.shape)}")
     fitted = not pages_per_split or not num_splits
     keep_first = int(keep_first) if window else 0
-    if (keep_first or chunk or distance is not None) and not fitted:
-        raise KernelError("attention_decode: kept first tokens, chunks and distance biases need shares fitted to the sequences")
+    if (keep_first or chunk or distance is not None or gate is not None) and not fitted:
+        raise KernelError("attention_decode: kept first tokens, chunks, distance biases and gates need shares fitted to the sequences")
     if fitted:
         pages_per_split, num_splits = decode_split(B, num_kv_heads, num_heads, page_table.shape[1])
     buf = scratch("attention_partials", (B * num_heads * num_splits * (head_dim + 2),), torch.float32)
@@ -1051,7 +1070,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, pa
             q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1],
             kv_len.data_ptr(), buf.data_ptr(), B, num_heads, num_kv_heads, head_dim, pages.shape[3], float(scale),
             int(window) if window else 0, num_splits, MIN_SHARE_PAGES, float(softcap or 0.0), _ptr(sinks),
-            1 if exact_weights else 0, keep_first, int(chunk or 0), dist_scale, dist_rate, _stream()))
+            1 if exact_weights else 0, keep_first, int(chunk or 0), dist_scale, dist_rate, gate_ptr, gate_ld, _stream()))
         return out
     _check(lib, lib.lp_attention_decode(
         q.data_ptr(), out.data_ptr(), pages.data_ptr(), page_table.data_ptr(), page_table.shape[1], kv_len.data_ptr(),
@@ -1119,25 +1138,26 @@ def attention_decode_fused(qkv: torch.Tensor, rotation: Rotation, out: torch.Ten
 def attention(ctx, q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, page_table: torch.Tensor, *,
               num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
               fast: bool, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None,
-              exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None) -> torch.Tensor:
+              exact_weights: bool = False, keep_first: int = 0, chunk: int = 0, distance=None, gate=None) -> torch.Tensor:
     """Attention of the step's tokens over the cache; picks the kernel for the step's shape. ``keep_first`` (with a
-    window): the first tokens of a sequence that stay visible beyond the window. ``chunk``, ``distance``: see
-    :func:`attention_plain`."""
+    window): the first tokens of a sequence that stay visible beyond the window. ``chunk``, ``distance``,
+    ``gate``: see :func:`attention_plain`."""
     tensor_cores = (fast and q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16
                     and head_dim % 16 == 0 and head_dim <= 256)
     keep_first = int(keep_first) if window else 0
     if tensor_cores and ctx.all_single:
         return attention_decode(q, out, pages, page_table, ctx.kv_len, ctx.buffer, num_heads=num_heads,
                                 num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale, window=window,
-                                softcap=softcap, sinks=sinks, exact_weights=exact_weights, keep_first=keep_first, chunk=chunk, distance=distance)
+                                softcap=softcap, sinks=sinks, exact_weights=exact_weights, keep_first=keep_first, chunk=chunk, distance=distance,
+                                gate=gate)
     if tensor_cores and not ctx.all_single:
         return attention_prefill(q, out, pages, page_table, ctx.q_start, ctx.kv_len, ctx.max_new,
                                  num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale,
                                  window=window, softcap=softcap, sinks=sinks, exact_weights=exact_weights,
-                                 keep_first=keep_first, chunk=chunk, distance=distance)
+                                 keep_first=keep_first, chunk=chunk, distance=distance, gate=gate)
     return attention_plain(q, out, pages, page_table, ctx.seq_ids, ctx.positions, num_heads=num_heads,
                            num_kv_heads=num_kv_heads, head_dim=head_dim, scale=scale, window=window, softcap=softcap,
-                           sinks=sinks, keep_first=keep_first, chunk=chunk, distance=distance)
+                           sinks=sinks, keep_first=keep_first, chunk=chunk, distance=distance, gate=gate)
 
 
 # --------------------------------------------------------------------------- latent attention
@@ -1784,7 +1804,7 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
                 num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, unit_norm_eps: Optional[float],
                 clear: Optional[torch.Tensor] = None, q_gain: Optional[torch.Tensor] = None,
                 k_gain: Optional[torch.Tensor] = None, gain_eps: float = 0.0, write_kv: bool = True,
-                value_norm_eps: Optional[float] = None) -> None:
+                value_norm_eps: Optional[float] = None, keep_values: Optional[torch.Tensor] = None, blend=None) -> None:
     """From the float32 projection ``qkv`` [T, H * dk + G * dk + G * dv]: add ``bias`` (float32, same width, or None),
     rotate queries and keys, divide each query and key head by its root mean square (``unit_norm_eps`` not None), and
     store queries to ``q_out`` [T, H * hdp] and keys and values into ``pages`` [num_pages, 2, G, page_size, hdp], every
@@ -1792,7 +1812,9 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
     before the rotation, query / key heads are RMS-normed over dk with that gain and ``gain_eps``. ``write_kv=False``:
     ``qkv`` [T, H * dk] holds queries only (a layer that attends over another layer's keys and values); ``pages`` only
     says how queries are stored. ``value_norm_eps``: every value head is divided by its root mean square over dv before it
-    is stored. ``qkv`` may be a column slice of a wider product."""
+    is stored. ``keep_values``: float32 [T, G * dv], receives this layer's values before they are stored. ``blend`` =
+    (first, share): values become (1 - share) * value + share * first with ``first`` float32 [T, G * dv] (an earlier layer's
+    ``keep_values``) and ``share`` one float32 number on the device. ``qkv`` may be a column slice of a wider product."""
     qkv_ptr, qkv_ld = _slice(qkv, "qkv_prepare qkv")
     _want(positions, "qkv_prepare positions", torch.int32, 1)
     _want(seq_ids, "qkv_prepare seq_ids", torch.int32, 1)
@@ -1819,6 +1841,13 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
         if bias.numel() != F:
             raise KernelError(f"qkv_prepare: a bias of {bias.numel()} values for {F} features")
     freq_ptr, rotary_dim, interleaved = rotation.checked("qkv_prepare")
+    for name, values in (("keep_values", keep_values), ("blend", None if blend is None else blend[0])):
+        if values is not None:
+            _want(values, f"qkv_prepare {name}", torch.float32, 2)
+            if values.shape != (T, G * dv):
+                raise KernelError(f"qkv_prepare: {name} {tuple(values.shape)} for {G} value heads of {dv}")
+    if blend is not None and _want(blend[1], "qkv_prepare share", torch.float32).numel() != 1:
+        raise KernelError("qkv_prepare: values are blended with one number")
     lib = library("elementwise")
     _check(lib, lib.lp_qkv_prepare(
         qkv_ptr, qkv_ld, _ptr(bias), freq_ptr, positions.data_ptr(), seq_ids.data_ptr(),
@@ -1826,7 +1855,8 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
         pages.data_ptr() if write_kv else None, _code(pages, "qkv_prepare pages"), T, H, G, dk, dv, hdp, rotary_dim, interleaved,
         0 if unit_norm_eps is None else 1, float(unit_norm_eps or 0.0), pages.shape[3], *_clear_args(clear, "qkv_prepare"),
         _ptr(q_gain), _ptr(k_gain) if write_kv else None, float(gain_eps), 0 if value_norm_eps is None else 1,
-        float(value_norm_eps or 0.0), _stream()))
+        float(value_norm_eps or 0.0), _ptr(keep_values), None if blend is None else blend[0].data_ptr(),
+        None if blend is None else blend[1].data_ptr(), _stream()))
 
 
 def post_norm_add(y: torch.Tensor, weight: torch.Tensor, eps: float, x: torch.Tensor, *, next_weight: Optional[torch.Tensor] = None,
@@ -2059,9 +2089,10 @@ def expert_scale(hidden: torch.Tensor, weights: torch.Tensor, expert_size: int, 
     return hidden
 
 
-def route_top(logits: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor, *, num_experts: int, top: int) -> torch.Tensor:
+def route_top(logits: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor, *, num_experts: int, top: int,
+              sigmoid: bool = False) -> torch.Tensor:
     """weights[t, e] for the E = ``num_experts`` experts: the ``top`` largest of logits[t, e] + bias[e] are chosen and
-    weighted by the softmax over the chosen logits alone (zero elsewhere). Columns of ``logits`` beyond E are gates of
+    weighted by the softmax over the chosen logits alone, or (``sigmoid``) by the sigmoid of each (zero elsewhere). Columns of ``logits`` beyond E are gates of
     experts that every token uses: weights[t, E + i] = sigmoid(logits[t, E + i]). ``logits``: float32 [T, E + extra]
     (may be a column slice); ``weights``: float32, same shape."""
     zp, ldz = _slice(logits, "route_top logits")
@@ -2075,8 +2106,85 @@ def route_top(logits: torch.Tensor, bias: Optional[torch.Tensor], weights: torch
             raise KernelError(f"route_top: a bias of {bias.numel()} values for {E} experts")
     lib = library("routing")
     _check(lib, lib.lp_route_top(zp, ldz, _ptr(bias), weights.data_ptr(), weights.shape[1], logits.shape[0], E, int(top),
-                                 logits.shape[1] - E, _stream()))
+                                 logits.shape[1] - E, 1 if sigmoid else 0, _stream()))
     return weights
+
+
+def expert_relu2(z: torch.Tensor, hidden: torch.Tensor, *, num_experts: int, expert_size: int, on_input: bool,
+                 weights: Optional[torch.Tensor] = None, top: int = 0, sigmoid: bool = False,
+                 clear: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Hidden activations of squared-ReLU experts from the float32 sums ``z`` of one stacked up product: column c belongs
+    to expert c // ``expert_size``; hidden[t, c] = max(w z, 0)^2 (``on_input``: the token's weight w multiplies the expert's
+    input) or w max(z, 0)^2. The weights are ``weights`` (float32 [T, >= E]) or, with ``top`` > 0, formed on the way from the
+    E logits that ``z`` then holds behind its E * expert_size sums: the ``top`` largest, weighted as in :func:`route_top`."""
+    zp, ldz = _slice(z, "expert_relu2 z")
+    _want(hidden, "expert_relu2 hidden", ndim=2)
+    E, F = int(num_experts), int(num_experts) * int(expert_size)
+    T = hidden.shape[0]
+    if hidden.shape[1] != F or z.shape != (T, F + (E if top > 0 else 0)):
+        raise KernelError(f"expert_relu2: sums {tuple(z.shape)}, hidden {tuple(hidden.shape)} for {E} experts of {expert_size}")
+    if (weights is None) == (top <= 0):
+        raise KernelError("expert_relu2: either weights or logits to choose from")
+    if weights is not None:
+        _want(weights, "expert_relu2 weights", torch.float32, 2)
+        if weights.shape[0] != T or weights.shape[1] < E:
+            raise KernelError(f"expert_relu2: weights {tuple(weights.shape)} for {T} tokens and {E} experts")
+    lib = library("routing")
+    _check(lib, lib.lp_expert_relu2(zp, ldz, hidden.data_ptr(), _code(hidden, "expert_relu2 hidden"), _ptr(weights),
+                                    0 if weights is None else weights.shape[1], T, E, int(expert_size), 1 if on_input else 0,
+                                    int(top), 1 if sigmoid else 0, *_clear_args(clear, "expert_relu2"), _stream()))
+    return hidden
+
+
+# --------------------------------------------------------------------------- a bundle of streams
+MAX_STREAMS = 32
+
+
+def stream_bundle(x: torch.Tensor, *, streams: int, y: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                  spread: Optional[torch.Tensor] = None, scale: float = 1.0, into: Optional[torch.Tensor] = None,
+                  gather: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  normed: Optional[torch.Tensor] = None, total: Optional[torch.Tensor] = None,
+                  clear: Optional[torch.Tensor] = None) -> None:
+    """What stands between two sublayers of a bundle of S = ``streams`` residual streams, in one pass.
+
+    ``x``: float32 [T, S, d], or [T, d] when all streams still equal that row. ``y`` (float32 [T, d], the finished sublayer's
+    result) enters them: x'_t = sum_s mix[s, t] x_s + scale * spread[t] * y (``mix`` float32 [S, S] indexed [from, to],
+    ``spread`` float32 [S]); ``into`` (float32 [T, S, d], may be ``x``) receives the new streams; without ``y`` they stay as
+    they are. With u = sum_s gather[s] x'_s (``gather`` float32 [S]; None: the plain sum), either the RMS norm of u
+    (``weight``, ``eps``) goes to ``normed`` [T, d] or u itself goes to ``total`` (float32 [T, d]; may be ``x`` when that is
+    [T, d])."""
+    S = int(streams)
+    _want(x, "stream_bundle x", torch.float32)
+    equal = x.dim() == 2
+    T, d = (x.shape[0], x.shape[-1])
+    if not equal and (x.dim() != 3 or x.shape[1] != S):
+        raise KernelError(f"stream_bundle: x {tuple(x.shape)} for {S} streams")
+    if not 1 <= S <= MAX_STREAMS:
+        raise KernelError(f"stream_bundle: {S} streams (at most {MAX_STREAMS})")
+
+    def check(t, name, shape):
+        if t is not None:
+            _want(t, f"stream_bundle {name}", torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"stream_bundle: {name} {tuple(t.shape)}, expected {shape}")
+    for t, name, shape in ((y, "y", (T, d)), (mix, "mix", (S, S)), (spread, "spread", (S,)), (into, "into", (T, S, d)),
+                           (gather, "gather", (S,)), (weight, "weight", (d,)), (total, "total", (T, d))):
+        check(t, name, shape)
+    if (weight is None) == (total is None) or (weight is None) != (normed is None):
+        raise KernelError("stream_bundle: the combination is either normed or stored as it is")
+    if normed is not None:
+        _want(normed, "stream_bundle normed", ndim=2)
+        if normed.shape != (T, d):
+            raise KernelError(f"stream_bundle: normed {tuple(normed.shape)} for {T} rows of {d}")
+    if y is not None and (mix is None or spread is None):
+        raise KernelError("stream_bundle: a result enters the streams through mix and spread")
+    if y is None and into is not None:
+        raise KernelError("stream_bundle: nothing enters the streams, so there are no new ones to store")
+    lib = library("stream_bundle")
+    _check(lib, lib.lp_stream_bundle(
+        x.data_ptr(), 1 if equal else 0, _ptr(y), _ptr(mix), _ptr(spread), float(scale), _ptr(into), _ptr(gather), _ptr(weight),
+        float(eps), _ptr(normed), F32 if normed is None else _code(normed, "stream_bundle normed"), _ptr(total), T, S, d,
+        *_clear_args(clear, "stream_bundle"), _stream()))
 
 
 def expert_act(z: torch.Tensor, weights: Optional[torch.Tensor], hidden: torch.Tensor, *, num_experts: int, expert_size: int,

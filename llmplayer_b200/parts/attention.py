@@ -50,6 +50,10 @@ class Attention(Part):
             raise ConfigError("a distance bias has a scale and a rate per head and comes with softmax weights at float32 precision")
         if s.value_norm_eps is not None and (s.shares_kv or not s.value_norm_eps > 0):
             raise ConfigError("normed values need keys and values of the layer's own and a positive constant")
+        if s.shares_kv and (s.shows_values or s.value_blend is not None):
+            raise ConfigError("a layer that attends over another layer's keys and values has no values to show or to blend")
+        if s.shows_values and s.value_blend is not None:
+            raise ConfigError("a layer either shows its values to later layers or blends an earlier layer's into its own")
         self.spec = spec
         self.position = POSITIONS.build(s.position)
         self.qkv: Optional[Linear] = None
@@ -62,6 +66,7 @@ class Attention(Part):
         self.q_gain: Optional[torch.Tensor] = None
         self.k_gain: Optional[torch.Tensor] = None
         self.output_bias: Optional[torch.Tensor] = None     # float32 [hidden]: what the output projection adds
+        self.blend: Optional[torch.Tensor] = None           # one float32 number: the share of the shown values
         self.distance = None                                # (scale, rate), float32 [heads] each
         self.inputs_stacked = False                         # set by an owner whose one product covers this part's inputs
         self._inputs = []
@@ -95,13 +100,17 @@ class Attention(Part):
         for name in (s.distance_scale, s.distance_rate):
             if name is not None:
                 specs[name] = TensorSpec((s.num_heads,), BIAS)
+        if s.value_blend is not None:
+            specs[s.value_blend] = TensorSpec((), BIAS)
+        if s.head_gate is not None:
+            specs[s.head_gate] = TensorSpec((s.num_heads, s.hidden_size), MATRIX)
         return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         super().load(tensors, runtime)
         s = self.spec
-        names = [s.q] if s.shares_kv else [s.q, s.k, s.v]
-        self._inputs = [tensors[n] for n in names]                   # rows: queries, keys, values
+        names = ([s.q] if s.shares_kv else [s.q, s.k, s.v]) + ([s.head_gate] if s.head_gate is not None else [])
+        self._inputs = [tensors[n] for n in names]                   # rows: queries, keys, values, the heads' gates
         if not self.inputs_stacked:
             self.qkv = Linear(self._inputs, runtime)
             self._inputs = []
@@ -126,6 +135,8 @@ class Attention(Part):
         self.q_gain = runtime.gain(tensors[s.q_norm]) if s.q_norm is not None else None
         self.k_gain = runtime.gain(tensors[s.k_norm]) if s.k_norm is not None else None
         self.output_bias = runtime.gain(tensors[s.o_bias]) if s.o_bias is not None else None
+        if s.value_blend is not None:
+            self.blend = runtime.gain(tensors[s.value_blend]).reshape(1)
         if s.distance_scale is not None:
             self.distance = (runtime.gain(tensors[s.distance_scale]), runtime.gain(tensors[s.distance_rate]))
 
@@ -178,7 +189,7 @@ class Attention(Part):
 
     def _forward_general(self, ctx, cache, x, residual: torch.Tensor, then_norm=None, overwrite: bool = False,
                          bias_later: bool = False) -> bool:
-        """A layer with biases, normed heads, capped scores, sinks, chunks, distance biases or values of another size than its keys:
+        """A layer with biases, normed heads, capped scores, sinks, chunks, distance biases, gated heads, blended values or values of another size than its keys:
         projection with float32 sums, one kernel that adds the biases, norms, rotates and stores queries, keys and
         values (heads padded to ``stored_dim``), then the attention kernels with the cap and the sinks as arguments.
         A layer that attends over another run's keys and values projects and prepares queries only."""
@@ -202,6 +213,10 @@ class Attention(Part):
         table = ctx.page_tables[cache.group_index]
         width = H * s.head_dim + (0 if s.shares_kv else G * (s.head_dim + self.value_dim))
         qkv = proj if offset == 0 and proj.shape[1] == width else proj[:, offset:offset + width]
+        gate = proj[:, offset + width:offset + width + H] if s.head_gate is not None else None
+        shown = None         # the values of the layer that shows them: the same tokens, so a buffer of the step and no cache
+        if s.shows_values or s.value_blend is not None:
+            shown = ctx.buffer("shown_values", (T, G * self.value_dim), torch.float32)
         q = ctx.buffer("q", (T, H * hd), rt.act_dtype)
         with ops.section("attention.position"):
             # an output product that sums partial results wants its target zero: this kernel clears it on the side
@@ -209,12 +224,14 @@ class Attention(Part):
             ops.qkv_prepare(qkv, self.bias, rotation, ctx.positions, ctx.seq_ids, table, q, cache.pages, num_heads=H,
                             num_kv_heads=G, key_dim=s.head_dim, value_dim=self.value_dim, unit_norm_eps=s.unit_norm_eps,
                             clear=clear, q_gain=self.q_gain, k_gain=self.k_gain, gain_eps=s.qk_norm_eps,
-                            write_kv=not s.shares_kv, value_norm_eps=s.value_norm_eps)
+                            write_kv=not s.shares_kv, value_norm_eps=s.value_norm_eps,
+                            keep_values=shown if s.shows_values else None,
+                            blend=(shown, self.blend) if s.value_blend is not None else None)
         o = ctx.buffer("attn_out", (T, H * hd), rt.act_dtype)
         with ops.section("attention.scores"):
             ops.attention(ctx, q, o, cache.pages, table, num_heads=H, num_kv_heads=G, head_dim=hd, scale=s.scale,
                           window=s.window, fast=rt.fast, softcap=s.softcap, sinks=self.sinks, exact_weights=s.exact_weights,
-                          keep_first=int(s.keep_first or 0), chunk=int(s.chunk or 0), distance=self.distance)
+                          keep_first=int(s.keep_first or 0), chunk=int(s.chunk or 0), distance=self.distance, gate=gate)
         with ops.section("attention.out"):
             if overwrite:
                 if clear is not None:

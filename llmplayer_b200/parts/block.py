@@ -17,7 +17,7 @@ from ..kernels import ops
 from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, FollowingNorm, Part, PendingNorm, Runtime
 from ..errors import ConfigError
 from .linear import Linear
-from .specs import BIAS, GAIN, MATRIX, BlockSpec, ParallelBlockSpec, PostNormBlockSpec, SandwichBlockSpec, TensorSpec
+from .specs import BIAS, GAIN, MATRIX, BlockSpec, BundleBlockSpec, ParallelBlockSpec, PostNormBlockSpec, SandwichBlockSpec, TensorSpec
 
 
 class PreNormBlock(Part):
@@ -451,6 +451,122 @@ class PostNormBlock(Part):
 _NO_CACHE = object()
 
 
+class BundleBlock(Part):
+    """Both sublayers on a bundle of S residual streams (hyper-connections): with u = sum_s gather[s] x_s and y =
+    F(norm(u)), every stream becomes x_t <- sum_s mix[s, t] x_s + residual_scale * spread[t] * y.
+
+    From outside the block keeps the contract of every other block, one stream [T, d] in, one out: the first of a row
+    of such blocks starts with S streams that all equal the stream it is handed (the copies are never written), each
+    hands the live bundle, in a buffer of the step [T, S, d], to the next, and the last one leaves the streams' sum in
+    the stream. Between two sublayers stands ONE kernel: it brings the finished sublayer's result into the streams and
+    norms the next sublayer's combination of the new ones on the way (and clears the buffer that the product after it
+    sums partial results into). The streams, the sublayers' results and the coefficients are float32."""
+
+    def __init__(self, spec: BundleBlockSpec):
+        self.spec = spec
+        if not 1 <= spec.streams <= ops.MAX_STREAMS:
+            raise ConfigError(f"{spec.streams} streams (supported: 1 to {ops.MAX_STREAMS})")
+        if len({spec.ffn is None, spec.ffn_norm is None, spec.ffn_connection is None}) != 1:
+            raise ConfigError("a feed-forward comes with the norm and the connection around it, or not at all")
+        self.mixer_norm = NORMS.build(spec.mixer_norm)
+        self.mixer = MIXERS.build(spec.mixer)
+        self.ffn_norm = NORMS.build(spec.ffn_norm) if spec.ffn is not None else None
+        self.ffn = FEED_FORWARDS.build(spec.ffn) if spec.ffn is not None else None
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and not getattr(norm, "fusable_rms", False):
+                raise ConfigError("the norms of a block with several streams are RMS norms")
+        self._mixer_stores = "overwrite" in inspect.signature(self.mixer.forward).parameters
+        self._ffn_stores = self.ffn is not None and "overwrite" in inspect.signature(self.ffn.forward).parameters
+        self._coefficients: Dict[str, torch.Tensor] = {}
+
+    kind_bundle = True
+
+    def children(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
+
+    @property
+    def capture_safe(self) -> bool:
+        return all(bool(getattr(part, "capture_safe", False)) for part in self.children())
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        out: Dict[str, TensorSpec] = {}
+        for part in self.children():
+            out.update(part.tensor_specs())
+        S = self.spec.streams
+        for c in (self.spec.mixer_connection, self.spec.ffn_connection):
+            if c is not None:
+                out.update({c.gather: TensorSpec((S,), BIAS), c.spread: TensorSpec((S,), BIAS), c.mix: TensorSpec((S, S), BIAS)})
+        return out
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        super().load(tensors, runtime)
+        for part in self.children():
+            part.load(tensors, runtime)
+        for c in (self.spec.mixer_connection, self.spec.ffn_connection):
+            if c is not None:
+                self._coefficients.update({n: runtime.gain(tensors[n]) for n in (c.gather, c.spread, c.mix)})
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def bundle(self, ctx, tokens: int) -> torch.Tensor:
+        """The step's buffer of streams, float32 [T, S, d]."""
+        return ctx.buffer("stream_bundle", (tokens, self.spec.streams, self.spec.mixer_norm.size), torch.float32)
+
+    def forward(self, ctx, cache, residual: torch.Tensor, normed_ready: bool = False, next_block=None) -> bool:
+        """``normed_ready``: the block before was of this kind; the bundle is live and this block's first norm is in the
+        shared "normed" buffer. ``next_block``: the block that runs next; if it is of this kind it is handed the bundle
+        with its first norm, else the streams' sum goes to ``residual``. Returns whether the bundle was handed on."""
+        s = self.spec
+        T = residual.shape[0]
+        h = ctx.buffer("normed", tuple(residual.shape), self.runtime.act_dtype)
+        y = ctx.buffer("sublayer_out", tuple(residual.shape), torch.float32)
+        bundle = self.bundle(ctx, T)
+        source = bundle if normed_ready else residual          # [T, d]: all streams still equal that row
+
+        def connect(finished, norm, connection, consumer) -> None:
+            """Bring the finished sublayer's result (None: there is none yet) into the streams; then the norm of the next
+            one's combination, or (no ``norm``) the streams' sum."""
+            nonlocal source
+            kw = {}
+            if finished is not None:
+                c = self._coefficients
+                kw = {"y": y, "mix": c[finished.mix], "spread": c[finished.spread], "scale": s.residual_scale}
+            with ops.section("norm"):
+                if norm is None:
+                    ops.stream_bundle(source, streams=s.streams, total=residual, **kw)
+                    return
+                clear = PreNormBlock._clear_for(ctx, consumer, T)
+                ops.stream_bundle(source, streams=s.streams, gather=connection, weight=norm.weight, eps=norm.spec.eps, normed=h,
+                                  into=bundle if finished is not None else None, clear=clear, **kw)
+                if clear is not None:
+                    ctx.note_cleared()
+            if finished is not None:
+                source = bundle
+
+        def run(part, stores, *args) -> None:
+            if stores:
+                part.forward(ctx, *args, h, y, overwrite=True)
+            else:
+                y.zero_()
+                part.forward(ctx, *args, h, y)
+
+        if not normed_ready:
+            connect(None, self.mixer_norm, self._coefficients[s.mixer_connection.gather], self.mixer)
+        run(self.mixer, self._mixer_stores, cache)
+        last = s.mixer_connection
+        if self.ffn is not None:
+            connect(last, self.ffn_norm, self._coefficients[s.ffn_connection.gather], self.ffn)
+            run(self.ffn, self._ffn_stores)
+            last = s.ffn_connection
+        if getattr(next_block, "kind_bundle", False) and next_block.spec.streams == s.streams:
+            connect(last, next_block.mixer_norm, next_block._coefficients[next_block.spec.mixer_connection.gather], next_block.mixer)
+            return True
+        connect(last, None, None, None)
+        return False
+
+
+BLOCKS.register("bundle", BundleBlock)
 BLOCKS.register("postnorm", PostNormBlock)
 BLOCKS.register("sandwich", SandwichBlock)
 BLOCKS.register("prenorm", PreNormBlock)

@@ -267,25 +267,36 @@ class Mixture(Part):
     by rows), whose hidden activations are multiplied by the token's weight for their expert, and ONE down product
     over the experts' down matrices stacked by columns, which sums the weighted outputs: every token passes through
     every expert, so the cost does not depend on the routing and the step has no host-side decisions (it replays
-    from a captured graph); what a token did not choose is multiplied by zero."""
+    from a captured graph); what a token did not choose is multiplied by zero.
+
+    Squared-ReLU experts have one up matrix each instead of gate and up: one stacked up product with float32 sums, then a
+    kernel that squares what is positive and applies the weights (to the expert's input or to its output). Where the
+    choice is by the largest logits, the router's rows are stacked below the up matrices and that kernel chooses as well:
+    the feed-forward is then two products with one kernel between them."""
     capture_safe = True
 
     def __init__(self, spec: MixtureSpec):
         s, r = spec, spec.routing
-        if r.scoring not in ("sigmoid_groups", "softmax_top", "softmax_groups"):
+        if r.scoring not in ("sigmoid_groups", "softmax_top", "softmax_groups", "sigmoid_top"):
             raise ConfigError(f"unknown scoring {r.scoring!r} of a router")
         if r.scoring != "softmax_groups" and (r.correction is not None or r.identity_experts or r.weight_scale != 1.0):
             raise ConfigError("a correction of the choice, identity experts and a constant on the weights belong to "
                               "scoring 'softmax_groups'")
         if r.identity_experts < 0:
             raise ConfigError(f"{r.identity_experts} identity experts")
-        if r.scoring == "softmax_groups" and (s.shared_size > 0 or s.activation != "silu"):
-            raise ConfigError("scoring 'softmax_groups' comes with silu experts and without a shared expert")
-        if s.activation not in ("silu", "clamped"):
+        if r.scoring == "softmax_groups" and (s.shared_size > 0 or s.activation == "clamped"
+                                              or (s.activation != "silu" and r.identity_experts)):
+            raise ConfigError("scoring 'softmax_groups' comes with silu experts (or squared-ReLU ones without identities) and "
+                              "without a shared expert")
+        if s.activation not in ("silu", "clamped", "relu2"):
             raise ConfigError(f"unknown activation {s.activation!r} of the experts")
         if s.activation == "clamped" and (not s.limit > 0 or (s.shared_size > 0 and not s.shared_limit > 0)):
             raise ConfigError(f"clamped experts need positive limits, got {s.limit} and {s.shared_limit}")
-        if r.scoring == "softmax_top" and (r.groups != 1 or r.keep_groups != 1):
+        if s.weight_on not in ("output", "input") or (s.weight_on == "input" and s.activation != "relu2"):
+            raise ConfigError(f"weights on {s.weight_on!r}: the weight multiplies an expert's output, or the input of a squared-ReLU expert")
+        if s.activation == "relu2" and s.shared_size > 0:
+            raise ConfigError("squared-ReLU experts come without a shared expert")
+        if r.scoring in ("softmax_top", "sigmoid_top") and (r.groups != 1 or r.keep_groups != 1):
             raise ConfigError("a router that takes the largest logits has no groups")
         if r.router_bias is not None and r.scoring != "softmax_top":
             raise ConfigError("only a router that takes the largest logits adds a bias to them")
@@ -305,7 +316,9 @@ class Mixture(Part):
         self.spec = spec
         self.router: Optional[Linear] = None
         self.gate_up: Optional[Linear] = None
+        self.up: Optional[Linear] = None
         self.down: Optional[Linear] = None
+        self.stacked_router = False
 
     def _experts(self):
         s = self.spec
@@ -318,7 +331,8 @@ class Mixture(Part):
         s = self.spec
         out: Dict[str, TensorSpec] = {}
         for prefix, size in self._experts():
-            out[prefix + "gate"] = TensorSpec((size, s.hidden_size), MATRIX)
+            if s.activation != "relu2":
+                out[prefix + "gate"] = TensorSpec((size, s.hidden_size), MATRIX)
             out[prefix + "up"] = TensorSpec((size, s.hidden_size), MATRIX)
             out[prefix + "down"] = TensorSpec((s.hidden_size, size), MATRIX)
         out[s.routing.router] = TensorSpec((s.routing.num_experts + s.routing.identity_experts, s.hidden_size), MATRIX)
@@ -332,24 +346,56 @@ class Mixture(Part):
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         super().load(tensors, runtime)
-        s = self.spec
+        s, r = self.spec, self.spec.routing
         experts = self._experts()
-        gate = torch.cat([tensors[p + "gate"] for p, _ in experts], dim=0)
         up = torch.cat([tensors[p + "up"] for p, _ in experts], dim=0)
         down = torch.cat([tensors[p + "down"] for p, _ in experts], dim=1).contiguous()
-        self.total = gate.shape[0]
+        self.total = up.shape[0]
+        self.down = Linear([down], runtime)
+        self.stacked_router = s.activation == "relu2" and r.scoring == "sigmoid_top"
+        if self.stacked_router:
+            self.up = Linear([up, tensors[r.router]], runtime)             # rows: the experts' up matrices, then the router
+            return
         # the shared expert's gate is one more row of the router's product
         self.router = Linear([tensors[s.routing.router]] + ([tensors[s.shared_gate]] if s.shared_gate is not None else []),
                              runtime)
         self.router_bias = runtime.gain(tensors[s.routing.router_bias]) if s.routing.router_bias is not None else None
         self.correction = runtime.gain(tensors[s.routing.correction]) if s.routing.correction is not None else None
+        if s.activation == "relu2":
+            self.up = Linear([up], runtime)
+            return
         # silu experts: the gated product applies the activation itself; clamped ones: float32 sums, then a kernel
+        gate = torch.cat([tensors[p + "gate"] for p, _ in experts], dim=0)
         self.gate_up = Linear([gate, up], runtime, gated=s.activation == "silu")
-        self.down = Linear([down], runtime)
 
     def buffer_to_clear(self, ctx, tokens: int):
         from ..kernels import ops
+        if self.stacked_router:
+            return self.up.sums_into(ctx, tokens, "ffn_up", ops.STORE)
         return self.router.sums_into(ctx, tokens, "router_logits", ops.STORE)
+
+    def _forward_stacked(self, ctx, x, residual: torch.Tensor, overwrite: bool) -> bool:
+        """Squared-ReLU experts chosen by their largest logits: sums and logits in one product, choice, weights and
+        activation in one kernel, one down product."""
+        from ..kernels import ops
+        s, r = self.spec, self.spec.routing
+        T = x.shape[0]
+        z = ctx.buffer("ffn_up", (T, self.up.out_features), torch.float32)
+        with ops.section("ffn.up"):
+            self.up.store(x, z, ctx)
+        h = ctx.buffer("ffn_hidden", (T, self.total), self.runtime.act_dtype)
+        clear = residual if overwrite and residual.dtype == torch.float32 and self.down.needs_zero(T) else None
+        with ops.section("ffn.act"):
+            ops.expert_relu2(z, h, num_experts=r.num_experts, expert_size=s.expert_size, on_input=s.weight_on == "input",
+                             top=r.top, sigmoid=True, clear=clear)
+        with ops.section("ffn.down"):
+            if clear is not None:
+                ctx.note_cleared()
+            if overwrite:
+                self.down.store(h, residual, ctx)
+            else:
+                self.down.accumulate(h, residual, ctx)
+        return False
 
     def forward(self, ctx, x, residual: torch.Tensor, overwrite: bool = False) -> bool:
         """Adds the mixture's output into ``residual`` (``overwrite``: stores it there instead)."""
@@ -357,14 +403,17 @@ class Mixture(Part):
         s, r = self.spec, self.spec.routing
         if isinstance(x, PendingNorm):
             x = x.tensor()
+        if self.stacked_router:
+            return self._forward_stacked(ctx, x, residual, overwrite)
         T = x.shape[0]
         columns = self.router.out_features              # the experts' logits (and the shared expert's gate)
         logits = ctx.buffer("router_logits", (T, columns), torch.float32)
         with ops.section("ffn.router"):
             self.router.store(x, logits, ctx)
             weights = ctx.buffer("router_weights", (T, columns), torch.float32)
-            if r.scoring == "softmax_top":
-                ops.route_top(logits, self.router_bias, weights, num_experts=r.num_experts, top=r.top)
+            if r.scoring in ("softmax_top", "sigmoid_top"):
+                ops.route_top(logits, self.router_bias, weights, num_experts=r.num_experts, top=r.top,
+                              sigmoid=r.scoring == "sigmoid_top")
             elif r.scoring == "softmax_groups":
                 ops.route_softmax(logits, self.correction, weights, groups=r.groups, keep=r.keep_groups, top=r.top,
                                   scale=r.weight_scale)
@@ -373,7 +422,14 @@ class Mixture(Part):
         h = ctx.buffer("ffn_hidden", (T, self.total), self.runtime.act_dtype)
         clear = residual if overwrite and residual.dtype == torch.float32 and self.down.needs_zero(T) else None
         rides = False
-        if s.activation == "clamped":
+        if s.activation == "relu2":
+            z = ctx.buffer("ffn_up", (T, self.total), torch.float32)
+            with ops.section("ffn.up"):
+                self.up.store(x, z, ctx)
+            with ops.section("ffn.act"):
+                ops.expert_relu2(z, h, num_experts=r.num_experts, expert_size=s.expert_size, on_input=s.weight_on == "input",
+                                 weights=weights, clear=clear)
+        elif s.activation == "clamped":
             z = ctx.buffer("ffn_up", (T, 2 * self.total), torch.float32)
             with ops.section("ffn.gate_up"):
                 self.gate_up.store(x, z, ctx)

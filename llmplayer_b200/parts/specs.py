@@ -135,13 +135,20 @@ class AttentionSpec:
     distance_scale: Optional[str] = None
     distance_rate: Optional[str] = None
     value_norm_eps: Optional[float] = None   # every value head is divided by its root mean square (no gain) and cached so
+    # Values of the same token from an earlier layer of the step: the layer with ``shows_values`` leaves its values (with
+    # their bias) for later layers; a layer with ``value_blend`` (a tensor of one number, lambda) caches and attends over
+    # (1 - lambda) v + lambda v_shown instead of its own v. Both have the same number and size of value heads.
+    shows_values: bool = False
+    value_blend: Optional[str] = None
+    head_gate: Optional[str] = None      # matrix [heads, hidden]: head h's output is multiplied by sigmoid(head_gate x)_h
 
     @property
     def general(self) -> bool:
         return (bool(self.keep_first) or self.value_dim not in (None, self.head_dim) or any(b is not None for b in (self.q_bias, self.k_bias, self.v_bias))
                 or self.unit_norm_eps is not None or self.softcap is not None or self.sink is not None or self.exact_weights
                 or self.q_norm is not None or self.k_norm is not None or self.o_bias is not None or self.sink_value is not None
-                or self.chunk is not None or self.distance_scale is not None or self.value_norm_eps is not None)
+                or self.chunk is not None or self.distance_scale is not None or self.value_norm_eps is not None
+                or self.shows_values or self.value_blend is not None or self.head_gate is not None)
 
 
 @dataclass(frozen=True)
@@ -424,6 +431,9 @@ class ExpertRoutingSpec:
     ``scoring="softmax_top"``: the ``top`` experts with the largest logits router x + ``router_bias`` are chosen, and
     their weights are the softmax over the chosen logits alone (``groups`` and ``keep_groups`` stay 1).
 
+    ``scoring="sigmoid_top"``: the ``top`` experts with the largest logits router x are chosen, and their weights are the
+    sigmoids of their logits themselves, not renormalised (``groups`` and ``keep_groups`` stay 1).
+
     ``scoring="softmax_groups"``: scores softmax(router x) over all router outputs: the ``num_experts`` experts and
     ``identity_experts`` further ones without tensors whose output is their input. The choice is made on score +
     ``correction`` [all outputs]; a group's score is its largest choice score, the ``top`` largest choice scores inside
@@ -450,7 +460,11 @@ class MixtureSpec:
     ``activation="clamped"``: an expert is down(g * sigmoid(1.702 g) * (u + 1)) with g = min(gate x, limit) and
     u = clamp(up x, -limit, limit); ``limit`` belongs to the routed experts, ``shared_limit`` to the shared one.
     ``shared_gate``: a matrix [1, hidden]; the shared expert's output is multiplied by sigmoid(shared_gate x), one
-    number per token."""
+    number per token.
+
+    ``activation="relu2"``: experts without a gate, down(max(up x, 0)^2) (tensors up / down; no shared expert).
+    ``weight_on="input"`` (with those): a token's weight w multiplies the expert's input, so that its output is
+    down(max(up (w x), 0)^2), instead of the expert's output."""
     hidden_size: int
     expert_size: int
     routing: ExpertRoutingSpec
@@ -462,6 +476,7 @@ class MixtureSpec:
     limit: float = 0.0
     shared_limit: float = 0.0
     shared_gate: Optional[str] = None
+    weight_on: str = "output"
 
 
 @dataclass(frozen=True)
@@ -533,6 +548,32 @@ class PostNormBlockSpec:
     post_ffn_norm: Optional[NormSpec] = None
     ffn_scale: Optional[str] = None
     kind: str = "postnorm"
+
+
+@dataclass(frozen=True)
+class ConnectionSpec:
+    """How one sublayer is connected to a bundle of S streams (hyper-connections); names of float tensors ``gather`` [S],
+    ``spread`` [S] and ``mix`` [S, S], indexed [from, to]. The sublayer F reads u = sum_s gather[s] x_s, and with y =
+    F(norm(u)) every stream becomes x_t <- sum_s mix[s, t] x_s + residual_scale * spread[t] * y."""
+    gather: str
+    spread: str
+    mix: str
+
+
+@dataclass(frozen=True)
+class BundleBlockSpec:
+    """One layer on a bundle of ``streams`` residual streams instead of one, each sublayer with an RMS norm in front and a
+    :class:`ConnectionSpec` around it. A row of such blocks starts with ``streams`` copies of the stream that enters it
+    and leaves their sum. ``ffn`` may be None (then its norm and connection are None as well)."""
+    streams: int
+    mixer_norm: NormSpec
+    mixer: object
+    mixer_connection: ConnectionSpec
+    ffn_norm: Optional[NormSpec] = None
+    ffn: Optional[object] = None
+    ffn_connection: Optional[ConnectionSpec] = None
+    residual_scale: float = 1.0
+    kind: str = "bundle"
 
 
 @dataclass(frozen=True)
