@@ -7,6 +7,7 @@
     python bench.py --design zasitar [--size s|m|l] [--layers N]      (the Zasitar design beside Botuvik and Llama)
     python bench.py --design dopuvik [--size s|m|l] [--layers N]      (the Dopuvik design beside Zasitar and Llama)
     python bench.py --design vomotar [--size s|m|l] [--layers N]      (the Vomotar design beside Dopuvik and Llama)
+    python bench.py --design zotolix [--size s|m|l] [--layers N]      (the Zotolix design beside Botuvik and Llama)
 
 One "step" is one decode step of the whole batch. The default run has the Llama-3.2-1B shape, a batch of 8
 sequences with 512-token prompts in a cache sized for a context of 4096. Every figure comes from the library's
@@ -39,6 +40,9 @@ attention beside a recurrence), and Llama.
 ``--design zasitar`` does the same for the Zasitar design (time-mixing layers, sliding-window attention with normed
 heads and keys shared between layers, results normed behind the sublayers) beside Botuvik, the closest existing design
 (a matrix recurrence among attention layers with sinks, dense and routed feed-forwards), and Llama.
+``--design zotolix`` does the same for the Zotolix design (attention in chunks with blended values on a bundle of residual
+streams, squared-ReLU experts) beside Botuvik, the closest existing design (attention with additive vectors and unit-norm
+heads, experts chosen by sigmoid scores), and Llama.
 """
 from __future__ import annotations
 
@@ -278,6 +282,26 @@ def vomotar_config(size, layers):
             "layers": [dict(delta if i % 4 else pair, mlp=dense) for i in range(layers)]}
 
 
+ZOTOLIX_CHUNK, ZOTOLIX_STREAMS = 1024, 4       # chunks of half of the measured prompt
+
+
+def zotolix_config(size, layers):
+    """Attention in chunks of ZOTOLIX_CHUNK tokens in every layer (grouped as in the Llama beside it), gated heads and
+    unit-norm heads taking turns (rotation over half a head and over whole heads), values blended with the first layer's,
+    ZOTOLIX_STREAMS streams. Every feed-forward is routed: 8 experts of a quarter of the Botuvik's dense width, 2 chosen."""
+    width, heads, _, _, ff = HYBRID_SIZES[size]
+    hd = width // heads
+
+    def mixer(dims):
+        return {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "v_mix": True,
+                "mask": {"size": ZOTOLIX_CHUNK}, "rot": {"base": 500000.0, "dims": dims}}
+    routed = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 2}}
+    return {"architecture": "Zotolix", "vocab": 32000, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+            "streams": ZOTOLIX_STREAMS, "residual_mult": 0.5,
+            "layers": [{"type": "attention" if i % 2 else "attention_2", "mixer": mixer(hd if i % 2 else hd // 2), "mlp": routed}
+                       for i in range(layers)]}
+
+
 def compare_designs(args, peaks) -> int:
     import torch
     from llmplayer_b200 import Engine
@@ -294,10 +318,10 @@ def compare_designs(args, peaks) -> int:
     clocks = ClockSampler()
     clocks.start()
     botuvik, zasitar, dopuvik = args.design == "botuvik", args.design == "zasitar", args.design == "dopuvik"
-    vomotar = args.design == "vomotar"
+    vomotar, zotolix = args.design == "vomotar", args.design == "zotolix"
     title = {"botuvik": "Botuvik design beside Ramupel and ", "zasitar": "Zasitar design beside Botuvik and ",
              "ramupel": "Ramupel design beside ", "dopuvik": "Dopuvik design beside Zasitar and ",
-             "vomotar": "Vomotar design beside Dopuvik and "}[args.design]
+             "vomotar": "Vomotar design beside Dopuvik and ", "zotolix": "Zotolix design beside Botuvik and "}[args.design]
     out = {"metric": f"prefill and decode tok/s of the {title}Llama at equal size (bf16)", "impl": "ours",
            "layers": layers, "batch": batch, "prompt_len": prompt, "prefill_len": prefill_len, "peaks": peaks, "sizes": {}}
     try:
@@ -312,6 +336,8 @@ def compare_designs(args, peaks) -> int:
                 designs = [("dopuvik", dopuvik_config(size, layers)), ("zasitar", zasitar_config(size, layers)), designs[1]]
             if vomotar:
                 designs = [("vomotar", vomotar_config(size, layers)), ("dopuvik", dopuvik_config(size, layers)), designs[1]]
+            if zotolix:
+                designs = [("zotolix", zotolix_config(size, layers)), ("botuvik", botuvik_config(size, layers)), designs[1]]
             if args.only:
                 designs = [d for d in designs if d[0] in args.only.split(",")]
             for name, raw in designs:
@@ -374,12 +400,14 @@ def compare_designs(args, peaks) -> int:
                 }
                 del engine, profiled
                 torch.cuda.empty_cache()
-            row["rooflines"] = {} if zasitar or dopuvik or vomotar else hybrid_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len)
+            row["rooflines"] = {} if zasitar or dopuvik or vomotar or zotolix else hybrid_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len)
             if vomotar and "vomotar" in row:
                 row["rooflines"].update(vomotar_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
             if "dopuvik" in row:
                 row["rooflines"].update(dopuvik_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
-            if botuvik or zasitar:
+            if zotolix and "zotolix" in row:
+                row["rooflines"].update(zotolix_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
+            if (botuvik or zasitar or zotolix) and "botuvik" in row:
                 row["rooflines"].update(botuvik_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
             if zasitar:
                 row["rooflines"].update(zasitar_rooflines(size, layers, row, peaks, batch, prompt + 10, prefill_len))
@@ -581,6 +609,66 @@ def vomotar_rooflines(size, layers, row, peaks, batch, context, n):
     }
 
 
+def zotolix_rooflines(size, layers, row, peaks, batch, context, n):
+    """The Zotolix kernels beside their Botuvik and Llama twins (``botuvik_rooflines``): prompt kernels against the bf16
+    tensor peak, decode and elementwise kernels against the copy bandwidth. Chunked attention's work counts the keys of a
+    query's own chunk only."""
+    width, heads, _, _, ff = HYBRID_SIZES[size]
+    flops, gbs = peaks["bf16_tflops"] * 1e12, peaks["hbm_gbs"] * 1e9
+    hd, G, W, S = width // heads, max(1, heads // 4), ZOTOLIX_CHUNK, ZOTOLIX_STREAMS
+    rows = 8 * (ff // 4)
+
+    def frac(work, ms, count, peak):
+        return None if not ms or not count else work / (ms / count / 1e3) / peak
+
+    def prepare(qkv_row):            # reads the float32 projection, writes bfloat16 queries, keys and values
+        return n * qkv_row * (4 + 2)
+    seen = sum(i % W + 1 for i in range(n))                          # (query, key) pairs inside the chunks
+    pre, dec = row["zotolix"]["prefill_sections_ms"], row["zotolix"]["decode_sections_ms"]
+    qkv_row = (heads + 2 * G) * hd
+    out = {
+        "prefill zotolix attention in chunks, keys seen (of tensor peak)": frac(heads * seen * 4 * hd, pre.get("attention.scores"), layers, flops),
+        # reads and writes the streams, reads the sublayer's float32 result, writes the bfloat16 norm; the model's first and
+        # last of these touch one row where the others touch S (2 layers - 1 in between)
+        "prefill zotolix streams between sublayers (of copy bandwidth)": frac(
+            n * width * ((2 * layers - 1) * (2 * S * 4 + 4 + 2) + (4 + 2) + (S * 4 + 4 + 4) - S * 4 + 4), pre.get("norm"), 1, gbs),
+        "prefill zotolix heads prepared, values blended (of copy bandwidth)": frac(
+            prepare(qkv_row) + n * G * hd * 4, pre.get("attention.position"), layers, gbs),
+        "prefill zotolix expert up product, all experts (of tensor peak)": frac(2.0 * n * width * rows, pre.get("ffn.up"), layers, flops),
+        "prefill zotolix expert activation (of copy bandwidth)": frac(n * rows * (4 * 2 / 8 + 2), pre.get("ffn.act"), layers, gbs),
+        "prefill zotolix expert down product, all experts (of tensor peak)": frac(2.0 * n * width * rows, pre.get("ffn.down"), layers, flops),
+        "decode zotolix attention in chunks (of copy bandwidth)": frac(
+            batch * (context % W) * 2 * G * hd * 2, dec.get("attention.scores"), layers, gbs),
+        "decode zotolix expert up product (of copy bandwidth)": frac(rows * width * 2, dec.get("ffn.up"), layers, gbs),
+        "decode zotolix expert down product (of copy bandwidth)": frac(rows * width * 2, dec.get("ffn.down"), layers, gbs),
+        "decode zotolix streams between sublayers (of copy bandwidth)": frac(
+            batch * width * (2 * S * 4 + 4 + 2), dec.get("norm"), 2 * layers + 1, gbs),
+    }
+    b = row.get("botuvik")
+    if b is not None:
+        bpre, bdec = b["prefill_sections_ms"], b["decode_sections_ms"]
+        n_att, n_dense = sum(1 for i in range(layers) if i % 4), sum(1 for i in range(layers) if i % 2 == 0)
+        dense_rows, routed_rows = n_dense * ff, (layers - n_dense) * (8 * (ff // 4) + ff // 4)
+        out.update({
+            "prefill botuvik norm behind a sublayer (of copy bandwidth)": frac(n * width * (4 + 4 + 4 + 2), bpre.get("norm"), 2 * layers, gbs),
+            "prefill botuvik heads prepared (of copy bandwidth)": frac(prepare(qkv_row), bpre.get("attention.position"), n_att, gbs),
+            "prefill botuvik dense up product (of tensor peak)": frac(2.0 * n * width * ff, bpre.get("ffn.up"), n_dense, flops),
+            "prefill botuvik dense activation (of copy bandwidth)": frac(n * ff * (4 + 2), bpre.get("ffn.act"), n_dense, gbs),
+            "prefill botuvik down products (of tensor peak)": frac(2.0 * n * width * (dense_rows + routed_rows), bpre.get("ffn.down"), 1, flops),
+            "decode botuvik dense up product (of copy bandwidth)": frac(ff * width * 2, bdec.get("ffn.up"), n_dense, gbs),
+            "decode botuvik down products (of copy bandwidth)": frac((dense_rows + routed_rows) * width * 2, bdec.get("ffn.down"), 1, gbs),
+            "decode botuvik norm behind a sublayer (of copy bandwidth)": frac(
+                batch * width * (4 + 4 + 4 + 2), bdec.get("norm"), 2 * layers, gbs),
+        })
+    l = row.get("llama")
+    if l is not None:
+        out["prefill llama attention (of tensor peak)"] = frac(
+            heads * n * (n + 1) * 2 * hd, l["prefill_sections_ms"].get("attention.scores"), layers, flops)
+        out["decode llama attention (of copy bandwidth)"] = frac(
+            batch * context * 2 * G * hd * 2, l["decode_sections_ms"].get("attention.scores"), layers, gbs)
+    return out
+
+
 def spread(values):
     return {"median": statistics.median(values), "min": min(values), "max": max(values), "repeats": len(values)}
 
@@ -601,8 +689,8 @@ def main() -> int:
     ap.add_argument("--prefill-only", action="store_true",
                     help="measure only the 2,048-token prefill (small runs for profiling)")
     ap.add_argument("--profile", action="store_true", help="add the device time per section of the model walk")
-    ap.add_argument("--design", default="llama", choices=("llama", "ramupel", "botuvik", "zasitar", "dopuvik", "vomotar"),
-                    help="ramupel / botuvik / zasitar / dopuvik / vomotar: that design beside the closest others at equal size (another workload; see "
+    ap.add_argument("--design", default="llama", choices=("llama", "ramupel", "botuvik", "zasitar", "dopuvik", "vomotar", "zotolix"),
+                    help="ramupel / botuvik / zasitar / dopuvik / vomotar / zotolix: that design beside the closest others at equal size (another workload; see "
                          "the module text)")
     ap.add_argument("--size", default=None, choices=sorted(HYBRID_SIZES), help="with --design: one size only")
     ap.add_argument("--only", default=None, help="with --design: only these of the designs beside each other (comma-separated)")
@@ -616,7 +704,7 @@ def main() -> int:
     if args.gpus != 1:
         print(f"bench.py measures one GPU; --gpus {args.gpus} is not supported by this single-GPU library")
         return 2
-    if args.design in ("ramupel", "botuvik", "zasitar", "dopuvik", "vomotar"):
+    if args.design != "llama":
         return compare_designs(args, load_peaks())
     args.warmup = max(3, args.warmup)
     repeats = max(1, args.repeats)

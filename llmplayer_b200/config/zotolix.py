@@ -200,7 +200,7 @@ class ZotolixConfig(ArchitectureConfig):
             if layer.mixer.v_mix:
                 sizes = (layer.mixer.kv_heads, layer.mixer.vdim)
                 first = first if first is not None else sizes
-                if sizes[0] * sizes[1] != first[0] * first[1]:
+                if sizes != first:
                     raise ConfigError(f"layers[{i}].mixer: {sizes[0]} value heads of {sizes[1]} cannot be blended with {first[0]} of {first[1]}")
 
     # ------------------------------------------------------------------ writing

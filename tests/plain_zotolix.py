@@ -120,8 +120,19 @@ def squared_relu_expert(x, up, down):
     return torch.clamp(x @ up.T, min=0.0) ** 2 @ down.T
 
 
-def mixture(h, w, p, m):
-    g = expert_weights(h @ w[p + "router"].T, m["router"]["top"])
+def routing_gap(z, top):
+    """How clearly the choice is made: the smallest distance of a chosen logit from one that is not."""
+    if top == z.shape[-1]:
+        return float("inf")
+    s = z.sort(dim=-1, descending=True).values
+    return float((s[:, top - 1] - s[:, top]).min())
+
+
+def mixture(h, w, p, m, gaps=None):
+    z = h @ w[p + "router"].T
+    if gaps is not None:
+        gaps.append(routing_gap(z, m["router"]["top"]))
+    g = expert_weights(z, m["router"]["top"])
     out = torch.zeros_like(h)
     for e in range(m["router"]["experts"]):
         rows = (g[:, e] > 0).nonzero()[:, 0]
@@ -131,9 +142,9 @@ def mixture(h, w, p, m):
 
 
 # --------------------------------------------------------------------------- the model
-def forward(cfg, weights, tokens, dtype=torch.float64, rows=None, streams=None):
+def forward(cfg, weights, tokens, dtype=torch.float64, rows=None, streams=None, gaps=None):
     """Logits [len(rows), vocab] (every position by default). ``streams``: a list that receives the sum of the
-    streams after every layer."""
+    streams after every layer. ``gaps``: a list that receives how clearly every mixture chose."""
     w = {n: t.to(dtype) if t.is_floating_point() else t for n, t in weights.items()}
     eps, m, S = cfg["norm"]["eps"], cfg["residual_mult"], cfg["streams"]
     x = w["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"]
@@ -145,7 +156,7 @@ def forward(cfg, weights, tokens, dtype=torch.float64, rows=None, streams=None):
                       layer["type"], first_values)
         X = scatter_streams(X, w[p + "hc1.mix"], w[p + "hc1.out"], y, m)
         if layer["mlp"] is not None:
-            y = mixture(rms_norm(gather_streams(X, w[p + "hc2.in"]), w[p + "norm2"], eps), w, p + "mlp.", layer["mlp"])
+            y = mixture(rms_norm(gather_streams(X, w[p + "hc2.in"]), w[p + "norm2"], eps), w, p + "mlp.", layer["mlp"], gaps)
             X = scatter_streams(X, w[p + "hc2.mix"], w[p + "hc2.out"], y, m)
         if streams is not None:
             streams.append(X.sum(0))
