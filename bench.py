@@ -374,14 +374,13 @@ def compare_designs(args, peaks) -> int:
                 decode_ms = statistics.median(lap["device_ms"] / lap["steps"] for lap in laps)
                 engine.check()
                 end = time.time()
-                # sections: one prompt alone, then decode steps alone (profile mode: no graphs, no overlap)
-                slot = profiled.acquire()
-                profiled.step([(slot, long_prompt)], [[prefill_len - 1]])
-                profiled.release(slot)
-                profiled.profile_report(reset=True)
-                slot = profiled.acquire()
-                profiled.step([(slot, long_prompt)], [[prefill_len - 1]])
-                profiled.release(slot)
+                # sections: prompts alone, then decode steps alone (profile mode: no graphs, no overlap)
+                for i in range(6):                    # two to warm up, four that are reported
+                    if i == 2:
+                        profiled.profile_report(reset=True)
+                    slot = profiled.acquire()
+                    profiled.step([(slot, long_prompt)], [[prefill_len - 1]])
+                    profiled.release(slot)
                 pre = profiled.profile_report(reset=True)
                 slots = [profiled.acquire() for _ in ps]
                 profiled.step(list(zip(slots, ps)), [[prompt - 1]] * batch)

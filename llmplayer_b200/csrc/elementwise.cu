@@ -211,7 +211,7 @@ extern "C" int lp_rmsnorm(float* x, const void* add, int add_dtype, const int* r
 }
 
 // ---------------------------------------------------------------- rotation + cache write
-// One block per token of the fused projection output
+// From a token's row of the fused projection output
 //   qkv[t] = [ H query heads | G key heads | G value heads ] x head_dim   (float32).
 // Queries and keys: the first `rd` features of a head are rotated by
 // angle = float(position) * inv_freq[pair] (cosine and sine are formed once per token and
@@ -633,7 +633,7 @@ extern "C" int lp_advance(int* tokens, int* positions, int* kv_len, const int* s
 }
 
 // ---------------------------------------------------------------- queries, keys and values of a general attention layer
-// One block per token of the fused projection output
+// From a token's row of the fused projection output
 //   qkv[t] = [ H query heads x dk | G key heads x dk | G value heads x dv ]   (float32),
 // for layers whose heads need more than a rotation: an additive bias per feature (`bias`, optional), the rotation of
 // the first `rd` features of every query and key head (pairs (2i, 2i+1) or (i, i + rd/2); angle = float(position) *
@@ -647,105 +647,111 @@ extern "C" int lp_advance(int* tokens, int* positions, int* kv_len, const int* s
 // dv (`vnorm_eps` inside the root). G = 0 with `pages` null: a layer that has queries only. `vkeep` (optional, float32
 // [T, G * dv]): the values of this layer, with their bias, are left there for later layers of the step. `vfirst` (the same
 // buffer, in a later layer) with `vmix` (one number lambda): a value becomes (1 - lambda) v + lambda vfirst before it is stored.
+// A warp holds its head in registers (lane l: features l, l + 32, ... PER of them), so that all of a head's loads are in
+// flight together. `angles` (optional): (cos, sin) of every token and pair, formed once for the step (rope_angles_kernel);
+// without it every lane forms the ones it needs.
 constexpr int PREP_MAX = 256;
-template <typename TQ, typename TKV>
+template <int PER, typename TQ, typename TKV>
 __global__ void __launch_bounds__(256)
 qkv_prepare_kernel(const float* __restrict__ qkv, int ld, const float* __restrict__ bias, const float* __restrict__ inv_freq,
-                   const int* __restrict__ positions, const int* __restrict__ seq_ids, const int* __restrict__ page_table,
-                   int pt_stride, TQ* __restrict__ q_out, TKV* __restrict__ pages, int H, int G, int dk, int dv, int hdp,
-                   int rd, int interleaved, int unit, float unit_eps, int page_size, float* __restrict__ zero,
-                   long long zero_count, const float* __restrict__ qgain, const float* __restrict__ kgain, float gain_eps,
-                   int vnorm, float vnorm_eps, float* __restrict__ vkeep, const float* __restrict__ vfirst,
-                   const float* __restrict__ vmix) {
-    __shared__ float cs[PREP_MAX];
-    __shared__ float buf[8][PREP_MAX];
+                   const float2* __restrict__ angles, const int* __restrict__ positions, const int* __restrict__ seq_ids,
+                   const int* __restrict__ page_table, int pt_stride, TQ* __restrict__ q_out, TKV* __restrict__ pages, int T,
+                   int H, int G, int dk, int dv, int hdp, int rd, int interleaved, int unit, float unit_eps, int page_size,
+                   float* __restrict__ zero, long long zero_count, const float* __restrict__ qgain,
+                   const float* __restrict__ kgain, float gain_eps, int vnorm, float vnorm_eps, float* __restrict__ vkeep,
+                   const float* __restrict__ vfirst, const float* __restrict__ vmix) {
+    __shared__ float buf[8][PER * 32];
     lp_grid_release();
     lp_grid_wait();
     clear_on_the_side(zero, zero_count);
-    const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int heads = H + 2 * G;
+    const long long work = (long long)blockIdx.x * 8 + warp;
+    if (work >= (long long)T * heads) return;
+    const int t = (int)(work / heads), item = (int)(work - (long long)t * heads);
     const int pos = positions[t];
     const int half = rd >> 1;
-    for (int i = tid; i < half; i += blockDim.x) {
-        float s, c;
-        sincosf((float)pos * inv_freq[i], &s, &c);
-        cs[2 * i] = c;
-        cs[2 * i + 1] = s;
-    }
-    __syncthreads();
     const float* row = qkv + (long long)t * ld;
     const long long page = G > 0 ? page_table[(long long)seq_ids[t] * pt_stride + pos / page_size] : 0;
     const int r = pos % page_size;
-    for (int item = warp; item < H + 2 * G; item += 8) {
-        if (item < H + G) {
-            const int src = item * dk;               // query heads, then key heads, lie one after another
-            const float* gain = item < H ? qgain : kgain;
-            float pre = 1.0f;
-            if (gain) {
-                float s0 = 0.f;
-                for (int e = lane; e < dk; e += 32) {
-                    const float val = row[src + e] + (bias ? bias[src + e] : 0.f);
-                    s0 += val * val;
-                }
-                pre = 1.0f / sqrtf(lp_warp_sum(s0) / (float)dk + gain_eps);
-            }
-            float ss = 0.f;
-            for (int e = lane; e < dk; e += 32) {
-                float val = row[src + e] + (bias ? bias[src + e] : 0.f);
-                if (gain) val = val * pre * gain[e];
+    const bool rotated = item < H + G;           // a query or key head; query, key and value heads lie one after another
+    const int g = item - H - G;                  // which value head otherwise
+    const int src = rotated ? item * dk : (H + G) * dk + g * dv;
+    const int n = rotated ? dk : dv;
+    float v[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int e = lane + 32 * i;
+        v[i] = e < n ? row[src + e] + (bias ? bias[src + e] : 0.f) : 0.f;
+    }
+    auto squares = [&] {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) ss += v[i] * v[i];
+        return lp_warp_sum(ss);
+    };
+    float factor = 1.0f;
+    if (rotated) {
+        const float* gain = item < H ? qgain : kgain;
+        if (gain) {
+            const float pre = 1.0f / sqrtf(squares() / (float)dk + gain_eps);
+#pragma unroll
+            for (int i = 0; i < PER; ++i)
+                if (lane + 32 * i < dk) v[i] = v[i] * pre * gain[lane + 32 * i];
+        }
+        if (rd > 0) {
+#pragma unroll
+            for (int i = 0; i < PER; ++i)
+                if (lane + 32 * i < rd) buf[warp][lane + 32 * i] = v[i];
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                const int e = lane + 32 * i;
                 if (e < rd) {
                     int pair, partner;
                     bool first;
                     if (interleaved) { pair = e >> 1; first = !(e & 1); partner = e ^ 1; }
                     else { first = e < half; pair = first ? e : e - half; partner = first ? e + half : e - half; }
-                    float other = row[src + partner] + (bias ? bias[src + partner] : 0.f);
-                    if (gain) other = other * pre * gain[partner];
-                    const float c = cs[2 * pair], s = cs[2 * pair + 1];
-                    val = first ? val * c - other * s : val * c + other * s;
+                    const float other = buf[warp][partner];
+                    float c, s;
+                    if (angles) {
+                        const float2 a = angles[(long long)t * half + pair];
+                        c = a.x; s = a.y;
+                    } else {
+                        sincosf((float)pos * inv_freq[pair], &s, &c);
+                    }
+                    v[i] = first ? v[i] * c - other * s : v[i] * c + other * s;
                 }
-                buf[warp][e] = val;
-                ss += val * val;
-            }
-            ss = lp_warp_sum(ss);
-            const float factor = unit ? 1.0f / sqrtf(ss / (float)dk + unit_eps) : 1.0f;
-            __syncwarp();
-            if (item < H) {
-                TQ* dst = q_out + ((long long)t * H + item) * hdp;
-                for (int e = lane; e < hdp; e += 32) dst[e] = lp_from_float<TQ>(e < dk ? buf[warp][e] * factor : 0.f);
-            } else {
-                TKV* dst = pages + (((page * 2 + 0) * G + (item - H)) * page_size + r) * hdp;
-                for (int e = lane; e < hdp; e += 32) dst[e] = lp_from_float<TKV>(e < dk ? buf[warp][e] * factor : 0.f);
-            }
-            __syncwarp();
-        } else {
-            const int g = item - H - G;
-            const int src = (H + G) * dk + g * dv;
-            TKV* dst = pages + (((page * 2 + 1) * G + g) * page_size + r) * hdp;
-            float factor = 1.0f;
-            if (vnorm) {
-                float ss = 0.f;
-                for (int e = lane; e < dv; e += 32) {
-                    const float val = row[src + e] + (bias ? bias[src + e] : 0.f);
-                    ss += val * val;
-                }
-                factor = 1.0f / sqrtf(lp_warp_sum(ss) / (float)dv + vnorm_eps);
-            }
-            const float lambda = vfirst ? *vmix : 0.f;
-            const long long at = ((long long)t * G + g) * dv;            // this value head in the buffer of a step's first values
-            for (int e = lane; e < hdp; e += 32) {
-                float val = 0.f;
-                if (e < dv) {
-                    val = (row[src + e] + (bias ? bias[src + e] : 0.f)) * factor;
-                    if (vkeep) vkeep[at + e] = val;
-                    if (vfirst) val = (1.0f - lambda) * val + lambda * vfirst[at + e];
-                }
-                dst[e] = lp_from_float<TKV>(val);
             }
         }
+        if (unit) factor = 1.0f / sqrtf(squares() / (float)dk + unit_eps);
+    } else if (vnorm) {
+        factor = 1.0f / sqrtf(squares() / (float)dv + vnorm_eps);
+    }
+    if (item < H) {
+        TQ* dst = q_out + ((long long)t * H + item) * hdp;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i < hdp) dst[lane + 32 * i] = lp_from_float<TQ>(v[i] * factor);
+        return;
+    }
+    TKV* dst = pages + (((page * 2 + (rotated ? 0 : 1)) * G + (rotated ? item - H : g)) * page_size + r) * hdp;
+    const float lambda = !rotated && vfirst ? *vmix : 0.f;
+    const long long at = ((long long)t * G + g) * dv;                // this value head in the buffer of a step's first values
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int e = lane + 32 * i;
+        float val = v[i] * factor;
+        if (!rotated && e < dv) {
+            if (vkeep) vkeep[at + e] = val;
+            if (vfirst) val = (1.0f - lambda) * val + lambda * vfirst[at + e];
+        }
+        if (e < hdp) dst[e] = lp_from_float<TKV>(val);
     }
 }
 
-extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const float* inv_freq, const int* positions,
-                              const int* seq_ids, const int* page_table, int pt_stride, void* q_out, int q_dtype,
+extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const float* inv_freq, const float* angles,
+                              const int* positions, const int* seq_ids, const int* page_table, int pt_stride, void* q_out, int q_dtype,
                               void* pages, int kv_dtype, int T, int H, int G, int dk, int dv, int hdp, int rd,
                               int interleaved, int unit, float unit_eps, int page_size, float* zero, long long zero_count,
                               const float* qgain, const float* kgain, float gain_eps, int vnorm, float vnorm_eps,
@@ -753,19 +759,29 @@ extern "C" int lp_qkv_prepare(const float* qkv, int ld, const float* bias, const
     if (T <= 0) return 0;
     if (vfirst && !vmix) LP_REFUSE("qkv_prepare: first values without the share they get");
     if (H <= 0 || G < 0 || dk <= 0 || dv <= 0) LP_REFUSE("qkv_prepare: %d / %d heads of %d and %d", H, G, dk, dv);
-    if (hdp < dk || hdp < dv || dk > PREP_MAX) LP_REFUSE("qkv_prepare: heads of %d and %d stored in %d (at most %d)", dk, dv, hdp, PREP_MAX);
+    if (hdp < dk || hdp < dv || hdp > PREP_MAX) LP_REFUSE("qkv_prepare: heads of %d and %d stored in %d (at most %d)", dk, dv, hdp, PREP_MAX);
     if (rd < 0 || rd > dk || (rd & 1)) LP_REFUSE("qkv_prepare: rotary width %d for heads of %d", rd, dk);
     if (rd > 0 && !inv_freq) LP_REFUSE("qkv_prepare: a rotation without frequencies");
     if (ld < (H + G) * dk + G * dv) LP_REFUSE("qkv_prepare: rows of %d values for %d", ld, (H + G) * dk + G * dv);
     if (G > 0 && (page_size <= 0 || !pages)) LP_REFUSE("qkv_prepare: needs the pages of the cache");
     if (G == 0) page_size = 1;
-#define LP_LAUNCH_PREP(TQ, TKV)                                                                                       \
-    lp_launch(qkv_prepare_kernel<TQ, TKV>, T, 256, 0, stream, qkv, ld, bias, inv_freq, positions, seq_ids, page_table, \
-              pt_stride, (TQ*)q_out, (TKV*)pages, H, G, dk, dv, hdp, rd, interleaved, unit, unit_eps, page_size, zero,  \
-              zero_count, qgain, kgain, gain_eps, vnorm, vnorm_eps, vkeep, vfirst, vmix)
-    if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_LAUNCH_PREP(float, float);
-    else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_LAUNCH_PREP(__nv_bfloat16, __nv_bfloat16);
+    const long long blocks = ((long long)T * (H + 2 * G) + 7) / 8;
+    if (blocks > 0x7fffffffLL) LP_REFUSE("qkv_prepare: %d tokens of %d heads exceed the grid", T, H + 2 * G);
+#define LP_LAUNCH_PREP(PER, TQ, TKV)                                                                                     \
+    lp_launch(qkv_prepare_kernel<PER, TQ, TKV>, (unsigned)blocks, 256, 0, stream, qkv, ld, bias, inv_freq,                \
+              (const float2*)angles, positions, seq_ids, page_table, pt_stride, (TQ*)q_out, (TKV*)pages, T, H, G, dk, dv,  \
+              hdp, rd, interleaved, unit, unit_eps, page_size, zero, zero_count, qgain, kgain, gain_eps, vnorm, vnorm_eps, \
+              vkeep, vfirst, vmix)
+#define LP_PICK_PREP(TQ, TKV)                                       \
+    do {                                                            \
+        if (hdp <= 64) LP_LAUNCH_PREP(2, TQ, TKV);                  \
+        else if (hdp <= 128) LP_LAUNCH_PREP(4, TQ, TKV);            \
+        else LP_LAUNCH_PREP(8, TQ, TKV);                            \
+    } while (0)
+    if (q_dtype == LP_F32 && kv_dtype == LP_F32) LP_PICK_PREP(float, float);
+    else if (q_dtype == LP_BF16 && kv_dtype == LP_BF16) LP_PICK_PREP(__nv_bfloat16, __nv_bfloat16);
     else LP_REFUSE("qkv_prepare: dtype codes q=%d kv=%d", q_dtype, kv_dtype);
+#undef LP_PICK_PREP
 #undef LP_LAUNCH_PREP
     return lp_check_launch("qkv_prepare");
 }

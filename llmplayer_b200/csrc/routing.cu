@@ -195,8 +195,12 @@ route_top_kernel(const float* __restrict__ z, int ldz, const float* __restrict__
 // hidden = max(w z, 0)^2; else its output: hidden = w max(z, 0)^2. The weights come from `weights` [T, ldw], or (`top` > 0)
 // are formed here from the token's E router logits, which are columns E * ff .. of the same product: every block chooses
 // for its own token (choose_top without a bias), so that no kernel stands between the product and its activation.
-// A token per blockIdx.y (and every gridDim.y-th one after it); VEC: four columns per thread (rows on 16-byte boundaries,
-// expert sizes of a multiple of four).
+// A token per blockIdx.y (and every gridDim.y-th one after it); VEC: columns per thread (1, or 16 bytes of the output:
+// then rows start on 16-byte boundaries and expert sizes are multiples of VEC).
+__device__ __forceinline__ uint32_t pack2(float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
 template <typename TH, int VEC>
 __global__ void __launch_bounds__(256)
 expert_relu2_kernel(const float* __restrict__ z, int ldz, TH* __restrict__ hidden, const float* __restrict__ weights, int ldw,
@@ -220,22 +224,26 @@ expert_relu2_kernel(const float* __restrict__ z, int ldz, TH* __restrict__ hidde
             const int c = i * VEC;
             const float we = w[c / ff];
             const float in = on_input ? we : 1.0f, after = on_input ? 1.0f : we;
-            if constexpr (VEC == 4) {
-                float v[4] = {0.f, 0.f, 0.f, 0.f};
-                if (we != 0.f) {                         // an expert that was not chosen: its sums are not even read
-                    const float4 z4 = *reinterpret_cast<const float4*>(row + c);
-                    v[0] = z4.x; v[1] = z4.y; v[2] = z4.z; v[3] = z4.w;
+            if constexpr (VEC > 1) {
+                float v[VEC];
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) {
+                for (int k = 0; k < VEC; ++k) v[k] = 0.f;
+                if (we != 0.f) {                         // an expert that was not chosen: its sums are not even read
+#pragma unroll
+                    for (int k = 0; k < VEC; k += 4) {
+                        const float4 z4 = *reinterpret_cast<const float4*>(row + c + k);
+                        v[k] = z4.x; v[k + 1] = z4.y; v[k + 2] = z4.z; v[k + 3] = z4.w;
+                    }
+#pragma unroll
+                    for (int k = 0; k < VEC; ++k) {
                         const float r = fmaxf(in * v[k], 0.f);
                         v[k] = r * r * after;
                     }
                 }
                 if constexpr (sizeof(TH) == 2) {
-                    uint2 packed;
-                    *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v[0], v[1]);
-                    *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v[2], v[3]);
-                    *reinterpret_cast<uint2*>(hidden + t * total + c) = packed;
+                    uint4 packed;
+                    packed.x = pack2(v[0], v[1]); packed.y = pack2(v[2], v[3]); packed.z = pack2(v[4], v[5]); packed.w = pack2(v[6], v[7]);
+                    *reinterpret_cast<uint4*>(hidden + t * total + c) = packed;
                 } else {
                     *reinterpret_cast<float4*>(hidden + t * total + c) = make_float4(v[0], v[1], v[2], v[3]);
                 }
@@ -469,15 +477,18 @@ extern "C" int lp_expert_relu2(const float* z, int ldz, void* hidden, int dtype,
     if (dtype != LP_F32 && dtype != LP_BF16) LP_REFUSE("expert_relu2: dtype code %d", dtype);
     const size_t smem = (size_t)2 * E * sizeof(float);
     if (smem > 48 * 1024) LP_REFUSE("expert_relu2: %d experts need %zu bytes of shared memory", E, smem);
-    const bool vec = ff % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)hidden) & 15) == 0;
-    int bx = (E * ff / (vec ? 4 : 1) + 255) / 256;
-    if (bx > 64) bx = 64;
+    const int wide = dtype == LP_F32 ? 4 : 8;
+    const bool vec = ff % wide == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)hidden) & 15) == 0;
+    // every block of a token chooses its experts anew: no more blocks per token than fill the GPU
+    int bx = (E * ff / (vec ? wide : 1) + 255) / 256;
+    const int enough = (8 * lp_sm_count() + T - 1) / T;
+    if (bx > enough) bx = enough;
     const dim3 grid(bx, T < 65535 ? T : 65535);
 #define LP_EXPERT_RELU2(TH, V)                                                                                           \
     lp_launch(expert_relu2_kernel<TH, V>, grid, 256, smem, stream, z, ldz, (TH*)hidden, weights, ldw, T, E, ff, on_input, \
               top, form, zero, zero_count)
     if (dtype == LP_F32) { if (vec) LP_EXPERT_RELU2(float, 4); else LP_EXPERT_RELU2(float, 1); }
-    else { if (vec) LP_EXPERT_RELU2(__nv_bfloat16, 4); else LP_EXPERT_RELU2(__nv_bfloat16, 1); }
+    else { if (vec) LP_EXPERT_RELU2(__nv_bfloat16, 8); else LP_EXPERT_RELU2(__nv_bfloat16, 1); }
 #undef LP_EXPERT_RELU2
     return lp_check_launch("expert_relu2");
 }

@@ -11,8 +11,13 @@
 
 namespace {
 
-constexpr int BUNDLE_THREADS = 256;
 constexpr int BUNDLE_MAX = 32;          // streams at most
+// Threads per block: 256 when there are tokens enough to fill the GPU, twice that for a handful of tokens (a decode step,
+// where a block's own latency is what counts), if the registers of that many streams allow it.
+constexpr int bundle_threads_max(int sx) { return sx > 0 && sx <= 4 ? 512 : 256; }
+// At most 64 registers per thread for so few streams, half of the SM's warps resident: what is waited for are the loads, and
+// with the compiler's own choice (100 registers, a quarter of the warps) 2,048 rows of 1,024 took 26.6 us instead of 20.5.
+constexpr int bundle_blocks_min(int sx) { return sx > 0 && sx <= 4 ? 2 : 1; }
 
 struct BundleArgs {
     const float* src;                   // x: token t's stream s at src + t * src_token + s * src_stream
@@ -62,13 +67,13 @@ template <int W> __device__ __forceinline__ void store_piece(__nv_bfloat16* p, c
 // SX > 0: that many streams, coefficients in registers. SX == 0: a.S streams (at most BUNDLE_MAX), coefficients in shared
 // memory and the token's streams read once per new stream.
 template <int SX, typename TOUT, int W>
-__global__ void __launch_bounds__(BUNDLE_THREADS)
+__global__ void __launch_bounds__(bundle_threads_max(SX), bundle_blocks_min(SX))
 stream_bundle_kernel(const BundleArgs a) {
     extern __shared__ __align__(16) float u_row[];          // [d]: the combination, until its root mean square is known
     __shared__ float coeff[SX > 0 ? 1 : BUNDLE_MAX * BUNDLE_MAX + 2 * BUNDLE_MAX];
     __shared__ float scratch[32];
     const int S = SX > 0 ? SX : a.S;
-    const int tid = threadIdx.x;
+    const int tid = threadIdx.x, threads = blockDim.x;
     lp_grid_release();
     constexpr int R = SX > 0 ? SX : 1;
     float mix[R][R], out[R], in[R];
@@ -82,8 +87,8 @@ stream_bundle_kernel(const BundleArgs a) {
             for (int t = 0; t < SX; ++t) mix[s][t] = a.y ? a.mix[s * SX + t] : 0.f;
         }
     } else {
-        for (int i = tid; i < S * S; i += BUNDLE_THREADS) coeff[i] = a.y ? a.mix[i] : 0.f;
-        for (int i = tid; i < S; i += BUNDLE_THREADS) {
+        for (int i = tid; i < S * S; i += threads) coeff[i] = a.y ? a.mix[i] : 0.f;
+        for (int i = tid; i < S; i += threads) {
             coeff[S * S + i] = a.y ? a.scale * a.out[i] : 0.f;
             coeff[S * S + S + i] = a.in_next ? a.in_next[i] : 1.0f;
         }
@@ -97,7 +102,7 @@ stream_bundle_kernel(const BundleArgs a) {
     float* dst = a.dst ? a.dst + t * S * a.d : nullptr;
     const bool norms = a.weight != nullptr;
     float ss = 0.f;
-    for (int c = tid * W; c < a.d; c += BUNDLE_THREADS * W) {
+    for (int c = tid * W; c < a.d; c += threads * W) {
         Piece<W> u;
 #pragma unroll
         for (int i = 0; i < W; ++i) u.v[i] = 0.f;
@@ -168,7 +173,7 @@ stream_bundle_kernel(const BundleArgs a) {
     if (!norms) return;
     const float factor = 1.0f / sqrtf(lp_block_sum(ss, scratch) / (float)a.d + a.eps);
     TOUT* h = reinterpret_cast<TOUT*>(a.normed) + t * a.d;
-    for (int c = tid * W; c < a.d; c += BUNDLE_THREADS * W) {          // a thread reads back what it wrote itself
+    for (int c = tid * W; c < a.d; c += threads * W) {          // a thread reads back what it wrote itself
         Piece<W> u = load_piece<W>(u_row + c);
         const Piece<W> g = load_piece<W>(a.weight + c);
 #pragma unroll
@@ -188,18 +193,16 @@ template <typename K> int grant_smem(K kernel, size_t bytes) {
     return 0;
 }
 
-template <int SX, typename TOUT> int launch_bundle(const BundleArgs& a, int T, bool wide, cudaStream_t stream) {
+template <int SX, typename TOUT, int W> int launch_bundle_of(const BundleArgs& a, int T, cudaStream_t stream) {
     const size_t smem = a.weight ? (size_t)a.d * sizeof(float) : 0;
-    if (wide) {
-        const int rc = grant_smem(stream_bundle_kernel<SX, TOUT, 4>, smem);
-        if (rc) return rc;
-        lp_launch(stream_bundle_kernel<SX, TOUT, 4>, (unsigned)T, BUNDLE_THREADS, smem, stream, a);
-    } else {
-        const int rc = grant_smem(stream_bundle_kernel<SX, TOUT, 1>, smem);
-        if (rc) return rc;
-        lp_launch(stream_bundle_kernel<SX, TOUT, 1>, (unsigned)T, BUNDLE_THREADS, smem, stream, a);
-    }
+    const int rc = grant_smem(stream_bundle_kernel<SX, TOUT, W>, smem);
+    if (rc) return rc;
+    const int threads = T <= 2 * lp_sm_count() && a.d > 256 * W ? bundle_threads_max(SX) : 256;
+    lp_launch(stream_bundle_kernel<SX, TOUT, W>, (unsigned)T, threads, smem, stream, a);
     return lp_check_launch("stream_bundle");
+}
+template <int SX, typename TOUT> int launch_bundle(const BundleArgs& a, int T, bool wide, cudaStream_t stream) {
+    return wide ? launch_bundle_of<SX, TOUT, 4>(a, T, stream) : launch_bundle_of<SX, TOUT, 1>(a, T, stream);
 }
 
 template <typename TOUT> int pick_bundle(const BundleArgs& a, int T, bool wide, cudaStream_t stream) {

@@ -32,7 +32,7 @@ _SIGNATURES = {
         "lp_rope_cache_write": [_P, _I, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "lp_advance": [_P, _P, _P, _P, _I, _P],
         "lp_rope_angles": [_P, _P, _P, _I, _I, _P],
-        "lp_qkv_prepare": [_P, _I, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P,
+        "lp_qkv_prepare": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P,
                            ctypes.c_longlong, _P, _P, _F, _I, _F, _P, _P, _P, _P],
         "lp_pair_norm_add": [_P, _P, _F, _F, _P, _P, _F, _F, _P, _P, _F, _I, _P, _I, _I, _I, _P, ctypes.c_longlong, _P],
         "lp_post_norm_add": [_P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P, ctypes.c_longlong, _P, _P, _P],
@@ -974,6 +974,7 @@ def _check_attention(q, out, pages, page_table, H, G, hd, what):
         raise KernelError(f"{what}: pages {tuple(pages.shape)} do not fit {G} key heads of {hd}")
 
 
+ANGLE_TABLE_TOKENS = 128      # from so many tokens on a step's angles are formed once, in a table, and not by every layer
 tcgen05_attention = True      # tests switch it off to reach the mma.sync kernel at every size
 
 
@@ -1804,7 +1805,8 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
                 num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, unit_norm_eps: Optional[float],
                 clear: Optional[torch.Tensor] = None, q_gain: Optional[torch.Tensor] = None,
                 k_gain: Optional[torch.Tensor] = None, gain_eps: float = 0.0, write_kv: bool = True,
-                value_norm_eps: Optional[float] = None, keep_values: Optional[torch.Tensor] = None, blend=None) -> None:
+                value_norm_eps: Optional[float] = None, keep_values: Optional[torch.Tensor] = None, blend=None,
+                angles: Optional[torch.Tensor] = None) -> None:
     """From the float32 projection ``qkv`` [T, H * dk + G * dk + G * dv]: add ``bias`` (float32, same width, or None),
     rotate queries and keys, divide each query and key head by its root mean square (``unit_norm_eps`` not None), and
     store queries to ``q_out`` [T, H * hdp] and keys and values into ``pages`` [num_pages, 2, G, page_size, hdp], every
@@ -1814,7 +1816,8 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
     says how queries are stored. ``value_norm_eps``: every value head is divided by its root mean square over dv before it
     is stored. ``keep_values``: float32 [T, G * dv], receives this layer's values before they are stored. ``blend`` =
     (first, share): values become (1 - share) * value + share * first with ``first`` float32 [T, G * dv] (an earlier layer's
-    ``keep_values``) and ``share`` one float32 number on the device. ``qkv`` may be a column slice of a wider product."""
+    ``keep_values``) and ``share`` one float32 number on the device. ``angles``: the table that :func:`rope_angles` forms for these positions
+    and this rotation; without it the kernel forms what it needs itself. ``qkv`` may be a column slice of a wider product."""
     qkv_ptr, qkv_ld = _slice(qkv, "qkv_prepare qkv")
     _want(positions, "qkv_prepare positions", torch.int32, 1)
     _want(seq_ids, "qkv_prepare seq_ids", torch.int32, 1)
@@ -1848,9 +1851,11 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], rotation: Rotat
                 raise KernelError(f"qkv_prepare: {name} {tuple(values.shape)} for {G} value heads of {dv}")
     if blend is not None and _want(blend[1], "qkv_prepare share", torch.float32).numel() != 1:
         raise KernelError("qkv_prepare: values are blended with one number")
+    if angles is not None and _want(angles, "qkv_prepare angles", torch.float32, 3).shape != (T, rotary_dim // 2, 2):
+        raise KernelError(f"qkv_prepare: angles {tuple(angles.shape)} for {T} tokens and a rotary width of {rotary_dim}")
     lib = library("elementwise")
     _check(lib, lib.lp_qkv_prepare(
-        qkv_ptr, qkv_ld, _ptr(bias), freq_ptr, positions.data_ptr(), seq_ids.data_ptr(),
+        qkv_ptr, qkv_ld, _ptr(bias), freq_ptr, _ptr(angles), positions.data_ptr(), seq_ids.data_ptr(),
         page_table.data_ptr(), page_table.shape[1], q_out.data_ptr(), _code(q_out, "qkv_prepare q_out"),
         pages.data_ptr() if write_kv else None, _code(pages, "qkv_prepare pages"), T, H, G, dk, dv, hdp, rotary_dim, interleaved,
         0 if unit_norm_eps is None else 1, float(unit_norm_eps or 0.0), pages.shape[3], *_clear_args(clear, "qkv_prepare"),

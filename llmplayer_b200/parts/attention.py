@@ -218,6 +218,10 @@ class Attention(Part):
         if s.shows_values or s.value_blend is not None:
             shown = ctx.buffer("shown_values", (T, G * self.value_dim), torch.float32)
         q = ctx.buffer("q", (T, H * hd), rt.act_dtype)
+        angles = None
+        if rotation.rotary_dim and T >= ops.ANGLE_TABLE_TOKENS:
+            with ops.section("attention.angles"):
+                angles = ctx.angles(rotation)         # formed once per step, for all layers that rotate alike
         with ops.section("attention.position"):
             # an output product that sums partial results wants its target zero: this kernel clears it on the side
             clear = residual if overwrite and residual.dtype == torch.float32 and self.out.needs_zero(T) else None
@@ -225,6 +229,7 @@ class Attention(Part):
                             num_kv_heads=G, key_dim=s.head_dim, value_dim=self.value_dim, unit_norm_eps=s.unit_norm_eps,
                             clear=clear, q_gain=self.q_gain, k_gain=self.k_gain, gain_eps=s.qk_norm_eps,
                             write_kv=not s.shares_kv, value_norm_eps=s.value_norm_eps,
+                            angles=angles,
                             keep_values=shown if s.shows_values else None,
                             blend=(shown, self.blend) if s.value_blend is not None else None)
         o = ctx.buffer("attn_out", (T, H * hd), rt.act_dtype)

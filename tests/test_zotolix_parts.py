@@ -123,7 +123,12 @@ def test_values_are_shown_and_blended(dtype, H, G, dk, dv, rd, unit):
         assert float(kv[1, ..., dv:].abs().sum()) == 0.0 and float(pages[1].abs().sum()) == 0.0
         return q_out.view(T, H, hdp)[..., :dk], kv[0, ..., :dk], kv[1, ..., :dv]
     shown = torch.full((T, G * dv), float("nan"), device="cuda")
-    for kw, ref in ((dict(keep_values=shown), v), (dict(blend=(first.cuda(), lam.cuda())), P.blend_values(v, first.double().reshape(T, G, dv), 0.3))):
+    angles = None                                                  # a step's table of angles must give the same bits
+    if rd:
+        angles = ops.rope_angles(i32(pos), rotation, torch.empty(T, rd // 2, 2, device="cuda"))
+        assert all(torch.equal(a, b) for a, b in zip(run(), run(angles=angles)))
+    for kw, ref in ((dict(keep_values=shown, angles=angles), v),
+                    (dict(blend=(first.cuda(), lam.cuda())), P.blend_values(v, first.double().reshape(T, G, dv), 0.3))):
         got = run(**kw)
         for name, g, r in zip(("queries", "keys", "values"), got, (q, k, ref)):
             check_error(f"heads prepared, {name}, {dtype}", f"{H}/{G} x {dk} / {dv}, {list(kw)[0]}", rel(g, r), lim)
