@@ -455,7 +455,7 @@ class BundleBlock(Part):
     """Both sublayers on a bundle of S residual streams (hyper-connections): with u = sum_s gather[s] x_s and y =
     F(norm(u)), every stream becomes x_t <- sum_s mix[s, t] x_s + residual_scale * spread[t] * y.
 
-    From outside the block keeps the contract of every other block, one stream [T, d] in, one out: the first of a row
+    From outside the block looks like every other block, one stream [T, d] in, one out: the first of a row
     of such blocks starts with S streams that all equal the stream it is handed (the copies are never written), each
     hands the live bundle, in a buffer of the step [T, S, d], to the next, and the last one leaves the streams' sum in
     the stream. Between two sublayers stands ONE kernel: it brings the finished sublayer's result into the streams and
